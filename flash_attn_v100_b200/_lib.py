@@ -1,15 +1,14 @@
-"""ctypes binding of the C ABI declared in include/fa_b200.h.
+"""ctypes bindings of the C ABIs declared in include/fa_b200.h and include/fa_b200_hybrid.h.
 
-The library is loaded from the package directory.  There is no fallback: if
-`libfa_b200.so` is missing the import of any operator raises, with the build
-command in the message.
+The libraries are loaded from the package directory, each when an operator of it is first used.  There is no
+fallback: if a library is missing, the use of any of its operators raises, with the build command in the message.
 """
 from __future__ import annotations
 
 import ctypes
 import os
 
-from .build import LIB_PATH
+from .build import HYBRID_LIB_PATH, LIB_PATH
 
 _c = ctypes
 _vp, _i, _i64, _sz = _c.c_void_p, _c.c_int, _c.c_int64, _c.c_size_t
@@ -60,24 +59,50 @@ SIGNATURES = {
     "fa_qkv_rope_append_bf16": (_i, [_vp] * 13 + [_i, _i, _i, _i, _i, _c.c_float, _i64, _i, _vp]),
 }
 
+# every symbol include/fa_b200_hybrid.h declares
+_f = _c.c_float
+HYBRID_SIGNATURES = {
+    "fah_last_error": (_c.c_char_p, []),
+    "fah_residual_norm": (_i, [_vp, _vp, _vp, _vp, _vp, _i, _i, _vp, _vp, _i64, _i, _f, _i, _vp]),
+    "fah_gated_norm": (_i, [_vp, _vp, _i64, _vp, _vp, _i64, _i, _f, _i, _vp]),
+    "fah_clamped_glu": (_i, [_vp, _vp, _i64, _i, _f, _f, _f, _i, _vp]),
+    "fah_side_gate": (_i, [_vp, _vp, _vp, _i, _i64, _i, _vp, _i64, _i, _i, _vp]),
+    "fah_lightning": (_i, [_vp, _i64] + [_i] * 6 + [_vp, _vp, _i, _vp, _vp, _vp, _i, _i64, _vp, _vp, _i, _vp]),
+    "fah_latent_prep": (_i, [_vp, _i64] + [_i] * 6 + [_vp, _vp, _f] + [_vp] * 6 + [_i, _i, _vp, _i, _i, _vp, _vp, _i64, _vp, _i, _vp]),
+    "fah_rotate_heads": (_i, [_vp, _vp, _vp, _i64, _i, _i, _i, _i, _i, _vp]),
+    "fah_latent_attention": (_i, [_vp, _vp, _i, _i, _vp, _vp, _vp, _i, _i, _vp, _i, _i, _vp, _vp, _vp, _i64, _i, _i, _i, _f, _vp,
+                                  _i64, _vp, _i, _vp]),
+}
+
 _lib = None
+_hybrid_lib = None
+
+
+def _open(path: str, signatures) -> ctypes.CDLL:
+    if not os.path.exists(path):
+        raise RuntimeError(
+            f"{path} is missing: the CUDA library has not been built. "
+            "Run `python -m flash_attn_v100_b200.build` (needs nvcc); there is no CPU fallback.")
+    lib = ctypes.CDLL(path)
+    for name, (res, args) in signatures.items():
+        fn = getattr(lib, name)  # AttributeError if the symbol is not exported
+        fn.restype = res
+        fn.argtypes = args
+    return lib
 
 
 def load() -> ctypes.CDLL:
     global _lib
-    if _lib is not None:
-        return _lib
-    if not os.path.exists(LIB_PATH):
-        raise RuntimeError(
-            f"{LIB_PATH} is missing: the CUDA library has not been built. "
-            "Run `python -m flash_attn_v100_b200.build` (needs nvcc); there is no CPU fallback.")
-    lib = ctypes.CDLL(LIB_PATH)
-    for name, (res, args) in SIGNATURES.items():
-        fn = getattr(lib, name)  # AttributeError if the symbol is not exported
-        fn.restype = res
-        fn.argtypes = args
-    _lib = lib
-    return lib
+    if _lib is None:
+        _lib = _open(LIB_PATH, SIGNATURES)
+    return _lib
+
+
+def load_hybrid() -> ctypes.CDLL:
+    global _hybrid_lib
+    if _hybrid_lib is None:
+        _hybrid_lib = _open(HYBRID_LIB_PATH, HYBRID_SIGNATURES)
+    return _hybrid_lib
 
 
 def last_error() -> str:
@@ -87,3 +112,9 @@ def last_error() -> str:
 def check(rc: int) -> None:
     if rc != 0:
         raise RuntimeError(last_error() or f"fa_b200 call failed with status {rc}")
+
+
+def check_hybrid(rc: int) -> None:
+    if rc != 0:
+        raise RuntimeError(load_hybrid().fah_last_error().decode("utf-8", "replace") or
+                           f"fa_b200_hybrid call failed with status {rc}")

@@ -1,0 +1,37 @@
+// Decayed linear attention (see lightning.cu and lightning_chunk.cu).
+#pragma once
+#include <cuda_runtime.h>
+#include <stdint.h>
+
+namespace fa {
+namespace hybrid {
+
+struct LightningArgs {
+  const void* qkv;           // T [tokens, stride]; per token the H x dk queries, H x dk keys and H x dv values
+  long long stride;
+  int off_q, off_k, off_v;
+  int heads, dk, dv;
+  const float* decay;        // [heads]
+  float* state;              // [n_slots, heads, dk, dv]
+  int n_slots;
+  const int32_t* slots;      // [n_seq] state slot of every sequence
+  const int32_t* starts;     // [n_seq] position of the sequence's first token in this call (0: the state starts at zero)
+  const int32_t* cu;         // [n_seq + 1] token offsets, or null: sequence i has the one token i
+  int n_seq;
+  long long total;           // tokens
+  void* out;                 // T [tokens, heads * dv]
+  int* status;
+  float* seg_state;          // scratch of the segmented prompt kernel: [segments, heads, dk, dv]
+  const int32_t* seg_seq;    // [n_seg] sequence of every segment
+  const int32_t* seg_tok;    // [n_seg] first token of every segment
+  int n_seg, seg_len, max_seg_per_seq;
+};
+
+// Token-by-token kernel: any size, both types; prompts and decode steps.
+template <typename T> cudaError_t launch_lightning_scan(const LightningArgs& a, cudaStream_t s);
+// One token per sequence; dv a multiple of 4 and at most 1024.
+template <typename T> cudaError_t launch_lightning_decode(const LightningArgs& a, int sm_count, cudaStream_t s);
+bool lightning_decode_supported(const LightningArgs& a);
+
+}  // namespace hybrid
+}  // namespace fa

@@ -1,0 +1,216 @@
+"""Decoder whose layers each name their sequence mixer and feed-forward (`HybridConfig`).
+
+A layer run is x += mixer(norm1(x)); x += mlp(norm2(x)); x += rmsnorm(proj(gelu(gate x) * side[token])) — the last two only
+where the configuration has them.  The residual x is fp32 throughout; h, the activations and the cached rows are the
+model's type (bfloat16, or float32 with every product in 32 bits).  Matrix products go to cuBLAS through torch; everything
+between them is libfa_b200_hybrid.  An update of x is not applied by a kernel of its own: it is left pending and the next norm's
+kernel adds it.
+
+Mixers are classes with the same four members (see `LightningMixer`), looked up by the type of their spec; what a mixer keeps
+between calls is described by `store` and lives in `HybridCache.stores`, one entry per layer run.
+"""
+from __future__ import annotations
+
+from dataclasses import dataclass
+from typing import List, Optional
+
+import torch
+
+from .. import hybrid_ops as hops
+from ..kv_cache import BLOCK_SIZE, HybridCache
+from .config import HybridConfig, LatentAttentionSpec, LightningSpec
+from .model import GreedyHead, Segments
+
+GLU_ALPHA, GLU_SHIFT = 1.702, 1.0      # g sigmoid(1.702 g) (u + 1)
+
+
+@dataclass
+class Step:
+    """One pass over the packed tokens of a batch: whole prompts, portions of prompts, or one token per sequence."""
+    tokens: torch.Tensor                 # [T] int64
+    positions: torch.Tensor              # [T] int32, place in the token's sequence (= its cache slot)
+    starts: torch.Tensor                 # [n_seq] int32, position of the sequence's first token in this pass
+    cu: Optional[torch.Tensor]           # [n_seq + 1] int32; None: one token per sequence
+    tok_seq: torch.Tensor                # [T] int32, sequence of every token
+    state_rows: torch.Tensor             # [n_seq] int32, state slot of every sequence
+    block_table: torch.Tensor            # [n_seq, max_blocks] int32
+    lens: Optional[List[int]]            # host: new tokens per sequence (None: one each)
+    past: Optional[List[int]]            # host: cached tokens per sequence (prompts only)
+    status: torch.Tensor
+
+
+def linear(h, w):
+    return h @ w.t()
+
+
+class LightningMixer:
+    """Decayed linear attention; keeps a fp32 state per request."""
+
+    def __init__(self, spec: LightningSpec, w: dict, eps: float):
+        self.spec, self.w, self.eps = spec, w, eps
+
+    @staticmethod
+    def store(spec: LightningSpec):
+        return ("state", spec.heads, spec.dim, spec.vdim)
+
+    def rope_key(self):
+        return None
+
+    def run(self, h, store, step: Step, rope):
+        s, w = self.spec, self.w
+        z = linear(h, w["w_in"])                                     # q | k | v | output gate
+        o = hops.lightning(z, w["in_at"][:3], s.heads, s.dim, s.vdim, w["decay"], store, step.state_rows, step.starts, step.status,
+                           cu_seqlens=step.cu)
+        at = w["in_at"][3]
+        return linear(hops.gated_norm(o, z[:, at:at + s.heads * s.vdim], w["norm"], self.eps), w["w_out"])
+
+
+class LatentAttentionMixer:
+    """Attention on cached latent rows; keeps `kv_rank` + `rot_dim` elements per token."""
+
+    def __init__(self, spec: LatentAttentionSpec, w: dict, eps: float):
+        self.spec, self.w, self.eps = spec, w, eps
+
+    @staticmethod
+    def store(spec: LatentAttentionSpec):
+        return ("latent", spec.kv_rank + spec.rot_dim)
+
+    def rope_key(self):
+        return self.spec.rot_base, self.spec.rot_dim
+
+    def run(self, h, store, step: Step, rope):
+        s, w = self.spec, self.w
+        cos, sin = rope
+        T, H = h.size(0), s.heads
+        z = linear(h, w["w_in"])                                     # query latent | latent | shared key part | head gates
+        at = w["in_at"]
+        gate = z[:, at[3]:at[3] + H]
+        cq, _, _ = hops.latent_prep(z, at[0], s.q_rank, at[1], s.kv_rank, at[2], s.rot_dim, w["q_norm"], w["kv_norm"], self.eps, cos, sin,
+                                    store, step.block_table, step.tok_seq, step.positions, step.status)
+        q = linear(cq, w["w_uq"]).view(T, H, s.dim + s.rot_dim)
+        # scores and values in the latent space: q W_uk against the cached latents, the weighted latent times W_uv
+        q_abs = torch.empty((T, H, s.kv_rank), dtype=h.dtype, device=h.device)
+        torch.bmm(q[..., :s.dim].transpose(0, 1), w["w_uk"], out=q_abs.transpose(0, 1))
+        lat = hops.latent_attention(q_abs, q, s.dim, cos, sin, store, step.block_table, step.tok_seq, step.positions, gate, s.kv_rank,
+                                    s.rot_dim, s.scale, step.status)
+        o = torch.empty((T, H, s.vdim), dtype=h.dtype, device=h.device)
+        torch.bmm(lat.transpose(0, 1), w["w_uv"].transpose(1, 2), out=o.transpose(0, 1))
+        return linear(o.view(T, H * s.vdim), w["w_out"])
+
+
+MIXERS = {LightningSpec: LightningMixer, LatentAttentionSpec: LatentAttentionMixer}
+
+
+class HybridDecoder(GreedyHead):
+    """Single-GPU decoder with the interface `GenerationRunner` drives (see `TPDecoder`)."""
+
+    supports_portions = True     # a prompt may be prefilled in several passes
+
+    def __init__(self, cfg: HybridConfig, weights, device="cuda"):
+        cfg.validate()
+        self.cfg, self.w = cfg, weights
+        self.rank, self.world, self.group, self.comm = 0, 1, None, None
+        self.device = torch.device(device)
+        self.dtype = weights["embed"].dtype
+        self.vl = cfg.vocab_size
+        if self.device.type == "cuda":
+            # 32-bit products stay 32-bit, and the partial sums of a bfloat16 product are added up in 32 bits
+            torch.backends.cuda.matmul.allow_tf32 = False
+            torch.backends.cuda.matmul.allow_bf16_reduced_precision_reduction = False
+        self.mixers = [MIXERS[type(l.mixer)](l.mixer, lw, cfg.norm_eps) for l, lw in zip(cfg.layers, weights["layers"])]
+        self.runs = cfg.runs()
+        self._rope_f = {}
+        for m in self.mixers:
+            key = m.rope_key()
+            if key is not None and key not in self._rope_f:
+                base, dims = key
+                i = torch.arange(0, dims, 2, dtype=torch.float64)
+                self._rope_f[key] = (float(base) ** (-i / dims)).to(device=self.device, dtype=torch.float32)
+        self._iota = torch.arange(1, dtype=torch.int32, device=self.device)
+        self.layer_hook = None     # called with the residual after every layer run (inspection and tests)
+
+    # ---- what GenerationRunner asks for ----------------------------------------------------------------
+    def make_cache(self, max_batch: int, max_seq_len: int, num_blocks: int = 0) -> HybridCache:
+        specs = [self.mixers[i].store(self.cfg.layers[i].mixer) for i, _ in self.runs]
+        per_seq = (max_seq_len + BLOCK_SIZE - 1) // BLOCK_SIZE
+        return HybridCache(specs, num_blocks or max_batch * per_seq, max_batch, per_seq, self.device, self.dtype)
+
+    def check_errors(self) -> None:
+        """Raise if a kernel of this model recorded an error on the device (its cache holds the status word)."""
+
+    def _range(self, n):
+        if self._iota.numel() < n:
+            self._iota = torch.arange(n, dtype=torch.int32, device=self.device)
+        return self._iota[:n]
+
+    def rope_tables(self, positions):
+        """fp32 cos / sin [T, dims / 2] of every rotation the layers use."""
+        out = {}
+        for key, f in self._rope_f.items():
+            a = torch.outer(positions.float(), f)
+            out[key] = (a.cos(), a.sin())
+        return out
+
+    def forward(self, token_ids, positions, kv: HybridCache, block_table, slots, max_blocks, *, cu_seqlens=None, max_seqlen=0,
+                seq_lens_after=None, seg=None, state_rows=None, want=None, lens=None, past=None):
+        """Arguments as `TPDecoder.forward`, and: `state_rows` [n_seq] table rows of the sequences (default 0 .. n_seq - 1), `lens` /
+        `past` (prompts: new and cached tokens per sequence, on the host), `want` rows of the packed tokens whose hidden state is
+        returned (default: the last of every sequence)."""
+        n_seq = slots.numel()
+        seg = seg or Segments(capture=False)
+        prompt = cu_seqlens is not None
+        if prompt and lens is None:
+            c = cu_seqlens.tolist()
+            lens = [b - a for a, b in zip(c, c[1:])]
+        if prompt and past is None:
+            past = [int(p) for p in slots.tolist()]
+        rows = self._range(n_seq) if state_rows is None else state_rows
+        if prompt:
+            tok_seq = torch.repeat_interleave(torch.arange(n_seq, dtype=torch.int32),
+                                              torch.tensor(lens)).to(self.device, non_blocking=True)
+        else:
+            tok_seq = self._range(n_seq)
+        step = Step(token_ids, positions, slots, cu_seqlens, tok_seq, rows, block_table, lens, past, kv.status)
+        if prompt and want is None:
+            want = (cu_seqlens[1:] - 1).long()
+        out = {}
+        seg.run(lambda: out.update(hidden=self._pass(step, kv, want)))
+        return out["hidden"]
+
+    def _pass(self, step: Step, kv: HybridCache, want):
+        cfg, w, eps = self.cfg, self.w, self.cfg.norm_eps
+        T = step.tokens.numel()
+        x = torch.empty((T, cfg.width), dtype=torch.float32, device=self.device)
+        rope = self.rope_tables(step.positions)
+        pend = {}                                       # the update of x that the next norm applies
+        for r, (i, again) in enumerate(self.runs):
+            lw, mixer = w["layers"][i], self.mixers[i]
+            first = r == 0
+            emb = dict(embed=w["embed"], tokens=step.tokens, init=first) if first or again else {}
+            h = hops.residual_norm(x, lw["norm1"], eps, **pend, **emb)
+            pend = dict(delta=mixer.run(h, kv.stores[r], step, rope.get(mixer.rope_key())))
+            mlp = cfg.layers[i].mlp
+            if mlp is not None:
+                h = hops.residual_norm(x, lw["norm2"], eps, **pend)
+                pend = dict(delta=linear(hops.clamped_glu(linear(h, lw["w_gu"]), mlp.limit, GLU_ALPHA, GLU_SHIFT), lw["w_down"]))
+            if cfg.side_dim:
+                xt = hops.residual_norm(x, None, eps, **pend)
+                y = hops.side_gate(linear(xt, lw["side_gate"]), w["side_embed"], step.tokens, i * cfg.side_dim)
+                pend = dict(delta=linear(y, lw["side_proj"]), delta_w=lw["side_norm"])
+            if self.layer_hook is not None:
+                hops.residual_norm(x, None, eps, **pend, out=False)
+                pend = {}
+                self.layer_hook(x)
+        if want is not None:
+            if want.numel() == 0:
+                return torch.empty((0, cfg.width), dtype=self.dtype, device=self.device)
+            x = x[want].contiguous()
+            if "delta" in pend:
+                pend = dict(pend, delta=pend["delta"][want].contiguous())
+        return hops.residual_norm(x, w["final_norm"], eps, **pend)
+
+    def logits(self, hidden):
+        """fp32 logits; the output matrix is the embedding table."""
+        if hidden.dtype == torch.float32:
+            return hidden @ self.w["embed"].t()
+        return torch.mm(hidden, self.w["embed"].t(), out_dtype=torch.float32)

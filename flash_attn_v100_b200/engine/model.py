@@ -19,6 +19,7 @@ from typing import Optional
 import torch
 
 from .. import _lib, ops
+from ..kv_cache import PagedKVCache
 from .config import ModelConfig
 
 
@@ -26,7 +27,44 @@ def _p(t):
     return ctypes.c_void_p(t.data_ptr())
 
 
-class TPDecoder:
+class GreedyHead:
+    """Greedy sampling over a vocabulary sharded across the ranks; the model gives `logits`, `rank`, `world`, `vl`, `comm`
+    and `group`."""
+
+    def greedy_local(self, hidden):
+        """This rank's best (value, index) per sequence over its vocabulary shard, and the shard's logits."""
+        logits = self.logits(hidden)
+        val, idx = logits.max(dim=-1)
+        pair = torch.stack([val, (idx + self.rank * self.vl).float()], dim=-1).contiguous()   # indices < 2^24: exact
+        return pair, logits
+
+    def greedy_gather(self, pair, out=None):
+        """All-gather of the per-rank (value, index) pairs into `out` [world, B, 2] (allocated if None)."""
+        if out is None:
+            out = torch.empty((self.world,) + pair.shape, dtype=pair.dtype, device=pair.device)
+        if self.world == 1:
+            out[0].copy_(pair)
+        elif self.comm is not None and self.comm.owns(out):
+            self.comm.all_gather_into(out, pair)
+        else:
+            torch.distributed.all_gather_into_tensor(out, pair, group=self.group)
+        return out
+
+    @staticmethod
+    def greedy_select(gathered):
+        best = gathered[..., 0].argmax(dim=0)                              # first maximum = lowest rank on ties
+        return gathered[..., 1].gather(0, best.unsqueeze(0)).squeeze(0).long()
+
+    def greedy_token(self, hidden):
+        """argmax over the vocabulary sharded across ranks: local max / argmax, then an all-gather of the
+        (value, index) pairs (the reference's `allgather`, parallel/tensor_parallel.py:172-190)."""
+        pair, logits = self.greedy_local(hidden)
+        return self.greedy_select(self.greedy_gather(pair)), logits
+
+
+class TPDecoder(GreedyHead):
+    supports_portions = False    # prefill attends only to the prompt's own tokens: a prompt is one pass
+
     def __init__(self, cfg: ModelConfig, weights, rank: int = 0, world: int = 1, group=None, device="cuda"):
         cfg.validate(world)
         self.cfg, self.w, self.rank, self.world, self.group = cfg, weights, rank, world, group
@@ -52,6 +90,17 @@ class TPDecoder:
         self.lib = _lib.load()
         self.inv_freq = 1.0 / (cfg.rope_theta ** (torch.arange(0, cfg.head_dim, 2, dtype=torch.float32,
                                                                device=self.device) / cfg.head_dim))
+
+    def make_cache(self, max_batch: int, max_seq_len: int, num_blocks: int = 0) -> PagedKVCache:
+        per_seq = (max_seq_len + 15) // 16
+        return PagedKVCache(num_blocks=num_blocks or max_batch * per_seq, num_layers=self.cfg.num_layers,
+                            num_kv_heads=self.kl, head_dim=self.cfg.head_dim, max_batch=max_batch,
+                            max_blocks_per_seq=per_seq, device=self.device, dtype=self.attn_dtype)
+
+    def check_errors(self) -> None:
+        """Raise if a kernel of this model recorded an error on the device."""
+        ops.check_async_errors(self.device)
+        ops.check_prefill_errors(self.device)
 
     # ---- small wrappers over the C ABI -------------------------------------------------
     def _stream(self):
@@ -136,7 +185,7 @@ class TPDecoder:
 
     # ---- one decoder stack pass -------------------------------------------------------
     def _stages(self, token_ids, positions, kv, block_table, slots, max_blocks, cu_seqlens, max_seqlen,
-                seq_lens_after):
+                seq_lens_after, want=None):
         """The pass as closures over a shared state dict: `first`, per layer (`attention_half`, `mlp_half`),
         `last`.  After `attention_half` the row-parallel output st["o"] and after `mlp_half` st["delta"]
         still have to be summed over the ranks, unless st["peer"] is set: then the halves have already done
@@ -221,10 +270,10 @@ class TPDecoder:
 
         def last():
             if fused:                      # the last all-reduce has applied the final norm
-                st["hidden"] = st["h"]
+                st["hidden"] = st["h"] if want is None else st["h"][want]
                 return
-            if prefill:
-                idx = (cu_seqlens[1:] - 1).long()
+            if prefill or want is not None:
+                idx = want if want is not None else (cu_seqlens[1:] - 1).long()
                 x_last, d_last = st["x"][idx].contiguous(), st["delta"][idx].contiguous()
             else:
                 x_last, d_last = st["x"], st["delta"]
@@ -233,16 +282,20 @@ class TPDecoder:
         return st, first, layers, last
 
     def forward(self, token_ids, positions, kv, block_table, slots, max_blocks, *, cu_seqlens=None, max_seqlen=0,
-                seq_lens_after=None, seg=None):
+                seq_lens_after=None, seg=None, state_rows=None, want=None, lens=None, past=None):
         """token_ids [T] int64; positions [T] int32 (rotary position of every token).
         Prefill (cu_seqlens given): packed prompts, `slots` [batch] = first cache slot per sequence; returns the
         hidden state of the last token of every sequence.  Decode: one token per sequence, `slots` [B] = slot of
         the new token, `seq_lens_after` [B] = lengths including it (default: slots + 1); returns [B, hidden].
         `seg` (see `Segments`) receives the compute between two collectives as one unit, so that a decode
-        step can be replayed as a chain of CUDA graphs with the NCCL calls in between."""
+        step can be replayed as a chain of CUDA graphs with the NCCL calls in between.
+        `want`: rows of the packed tokens whose hidden state is returned instead.  `state_rows`, `lens` and `past` are for
+        models with per-request state or portioned prompts; this one has neither."""
+        if past is not None and any(past):
+            raise NotImplementedError("TPDecoder prefills a prompt in one pass")
         seg = seg or Segments(capture=False)
         st, first, layers, last = self._stages(token_ids, positions, kv, block_table, slots, max_blocks, cu_seqlens,
-                                               max_seqlen, seq_lens_after)
+                                               max_seqlen, seq_lens_after, want)
         seg.run(first)
         for attention_half, mlp_half in layers:
             seg.run(attention_half)
@@ -255,13 +308,13 @@ class TPDecoder:
         return st["hidden"]
 
     def forward_stages(self, token_ids, positions, kv, block_table, slots, max_blocks, *, cu_seqlens=None,
-                       max_seqlen=0, seq_lens_after=None):
+                       max_seqlen=0, seq_lens_after=None, state_rows=None, want=None, lens=None, past=None):
         """The same pass as a generator: it yields every tensor that has to be summed over the ranks (the
         caller all-reduces it in place before resuming) and finally returns the hidden state through
         StopIteration.  Several passes over independent token batches can thus be advanced in turn, each on
         its own stream, so that one batch's all-reduce overlaps the other's compute (`forward_overlapped`)."""
         st, first, layers, last = self._stages(token_ids, positions, kv, block_table, slots, max_blocks, cu_seqlens,
-                                               max_seqlen, seq_lens_after)
+                                               max_seqlen, seq_lens_after, want)
         first()
         for attention_half, mlp_half in layers:
             attention_half()
@@ -291,35 +344,9 @@ class TPDecoder:
                         live.remove(i)
         return out
 
-    def greedy_local(self, hidden):
-        """This rank's best (value, index) per sequence over its vocabulary shard, and the shard's logits."""
-        logits = (hidden @ self.w["lm_head"].t()).float()                 # [B, vocab/world]
-        val, idx = logits.max(dim=-1)
-        pair = torch.stack([val, (idx + self.rank * self.vl).float()], dim=-1).contiguous()   # indices < 2^24: exact
-        return pair, logits
-
-    def greedy_gather(self, pair, out=None):
-        """All-gather of the per-rank (value, index) pairs into `out` [world, B, 2] (allocated if None)."""
-        if out is None:
-            out = torch.empty((self.world,) + pair.shape, dtype=pair.dtype, device=pair.device)
-        if self.world == 1:
-            out[0].copy_(pair)
-        elif self.comm is not None and self.comm.owns(out):
-            self.comm.all_gather_into(out, pair)
-        else:
-            torch.distributed.all_gather_into_tensor(out, pair, group=self.group)
-        return out
-
-    @staticmethod
-    def greedy_select(gathered):
-        best = gathered[..., 0].argmax(dim=0)                              # first maximum = lowest rank on ties
-        return gathered[..., 1].gather(0, best.unsqueeze(0)).squeeze(0).long()
-
-    def greedy_token(self, hidden):
-        """argmax over the vocabulary sharded across ranks: local max / argmax, then an all-gather of the
-        (value, index) pairs (the reference's `allgather`, parallel/tensor_parallel.py:172-190)."""
-        pair, logits = self.greedy_local(hidden)
-        return self.greedy_select(self.greedy_gather(pair)), logits
+    def logits(self, hidden):
+        """This rank's vocabulary shard of the logits, fp32."""
+        return (hidden @ self.w["lm_head"].t()).float()                 # [B, vocab/world]
 
 
 class Segments:

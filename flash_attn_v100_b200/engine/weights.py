@@ -14,7 +14,7 @@ from typing import Dict, List
 
 import torch
 
-from .config import ModelConfig
+from .config import HybridConfig, LightningSpec, ModelConfig
 
 
 def _randn(shape, gen, std, device, dtype):
@@ -83,3 +83,115 @@ def make_rank_weights(cfg: ModelConfig, rank: int, world: int, seed: int, device
         "lm_head": glob["lm_head"][rank * vl:(rank + 1) * vl].contiguous().to(device),
         "final_ln": glob["final_ln"].to(device),
     }
+
+
+def rank_weights_from_tensors(cfg: ModelConfig, tensors: Dict[str, torch.Tensor], rank: int, world: int, device):
+    """The same per-rank dictionary from named full-size tensors: 'embed', 'lm_head', 'final_ln' and 'l<i>.<name>' with
+    the names of `make_full_layer`."""
+    cfg.validate(world)
+    layers = []
+    for l in range(cfg.num_layers):
+        pre = f"l{l}."
+        full = {k[len(pre):]: t.to(torch.bfloat16) for k, t in tensors.items() if k.startswith(pre)}
+        layers.append(shard_layer(cfg, full, rank, world, device))
+    vl = cfg.vocab_size // world
+    get = lambda n: tensors[n].to(torch.bfloat16)
+    return {"layers": layers, "embed": get("embed").to(device), "final_ln": get("final_ln").to(device),
+            "lm_head": get("lm_head")[rank * vl:(rank + 1) * vl].contiguous().to(device)}
+
+
+# ---- hybrid decoders -------------------------------------------------------------------------------------------
+def hybrid_tensor_shapes(cfg: HybridConfig) -> Dict[str, tuple]:
+    """Name and shape of every tensor of the model."""
+    W = cfg.width
+    out = {"embed": (cfg.vocab_size, W), "final.norm": (W,)}
+    if cfg.side_dim:
+        out["side.embed"] = (cfg.vocab_size, len(cfg.layers) * cfg.side_dim)
+    for i, layer in enumerate(cfg.layers):
+        m, pre = layer.mixer, f"l{i}."
+        out[pre + "norm1"] = (W,)
+        if isinstance(m, LightningSpec):
+            kd, vd = m.heads * m.dim, m.heads * m.vdim
+            mix = {"q": (kd, W), "k": (kd, W), "v": (vd, W), "g": (vd, W), "o": (W, vd), "norm": (vd,)}
+        else:
+            H = m.heads
+            mix = {"dq": (m.q_rank, W), "dq.norm": (m.q_rank,), "uq": (H * (m.dim + m.rot_dim), m.q_rank),
+                   "dkv": (m.kv_rank + m.rot_dim, W), "dkv.norm": (m.kv_rank,), "uk": (H * m.dim, m.kv_rank),
+                   "uv": (H * m.vdim, m.kv_rank), "g": (H, W), "o": (W, H * m.vdim)}
+        out.update({pre + "mix." + k: s for k, s in mix.items()})
+        if layer.mlp is not None:
+            F = layer.mlp.ff
+            out.update({pre + "norm2": (W,), pre + "mlp.gate": (F, W), pre + "mlp.up": (F, W), pre + "mlp.down": (W, F)})
+        if cfg.side_dim:
+            out.update({pre + "side.gate": (cfg.side_dim, W), pre + "side.proj": (W, cfg.side_dim), pre + "side.norm": (W,)})
+    return out
+
+
+def random_hybrid_tensors(cfg: HybridConfig, seed: int, device="cpu", dtype=torch.bfloat16) -> Dict[str, torch.Tensor]:
+    """Seeded random tensors: matrices N(0, 1 / inputs), norm weights 1 + N(0, 0.1^2), embeddings N(0, 1)."""
+    g = torch.Generator(device=device).manual_seed(seed)
+    out = {}
+    for name, shape in hybrid_tensor_shapes(cfg).items():
+        t = torch.randn(shape, generator=g, device=device)
+        if len(shape) == 1:
+            t = 1.0 + 0.1 * t
+        elif not name.endswith("embed"):
+            t = t / shape[1] ** 0.5
+        out[name] = t.to(dtype)
+    return out
+
+
+def _stack(mats, multiple: int = 8):
+    """Several [n_i, inputs] matrices as one, every block padded with zero rows to a multiple of `multiple` (so that the
+    columns of the product stay 16-byte aligned); returns the matrix and the first row of every block."""
+    rows, at, n = [], [], 0
+    for w in mats:
+        at.append(n)
+        pad = -w.size(0) % multiple
+        rows.append(w)
+        if pad:
+            rows.append(torch.zeros((pad, w.size(1)), dtype=w.dtype, device=w.device))
+        n += w.size(0) + pad
+    return torch.cat(rows).contiguous(), tuple(at)
+
+
+def hybrid_weights(cfg: HybridConfig, tensors: Dict[str, torch.Tensor], dtype, device):
+    """The model's tensors in the layout the decoder runs: projections of the same input stacked into one matrix.
+    {'embed', 'side_embed', 'final_norm', 'layers': [dict per layer]}."""
+    want = hybrid_tensor_shapes(cfg)
+    missing, extra = sorted(set(want) - set(tensors)), sorted(set(tensors) - set(want))
+    if missing or extra:
+        raise ValueError(f"tensors do not fit the configuration: missing {missing[:5]}, unknown {extra[:5]}")
+    for name, shape in want.items():
+        if tuple(tensors[name].shape) != shape:
+            raise ValueError(f"{name} has shape {tuple(tensors[name].shape)}, the configuration says {shape}")
+
+    def get(name):
+        return tensors[name].to(device=device, dtype=dtype).contiguous()
+
+    layers = []
+    for i, layer in enumerate(cfg.layers):
+        m, pre = layer.mixer, f"l{i}."
+        mix = lambda n: get(pre + "mix." + n)
+        lw = {"norm1": get(pre + "norm1")}
+        if isinstance(m, LightningSpec):
+            lw["w_in"], lw["in_at"] = _stack([mix(n) for n in ("q", "k", "v", "g")])
+            lw["norm"], lw["w_out"] = mix("norm"), mix("o")
+            lw["decay"] = torch.tensor(m.decay, dtype=torch.float32, device=device)
+        else:
+            dkv = mix("dkv")
+            lw["w_in"], lw["in_at"] = _stack([mix("dq"), dkv[:m.kv_rank], dkv[m.kv_rank:], mix("g")])
+            lw["q_norm"], lw["kv_norm"], lw["w_uq"], lw["w_out"] = mix("dq.norm"), mix("dkv.norm"), mix("uq"), mix("o")
+            uk, uv = mix("uk"), mix("uv")
+            lw["w_ukv"] = torch.cat([uk, uv]).contiguous()             # expansion of the latents (prompts)
+            lw["w_uk"] = lw["w_ukv"][:m.heads * m.dim].view(m.heads, m.dim, m.kv_rank)       # per head (decode)
+            lw["w_uv"] = lw["w_ukv"][m.heads * m.dim:].view(m.heads, m.vdim, m.kv_rank)
+        if layer.mlp is not None:
+            lw["norm2"] = get(pre + "norm2")
+            lw["w_gu"] = torch.cat([get(pre + "mlp.gate"), get(pre + "mlp.up")]).contiguous()
+            lw["w_down"] = get(pre + "mlp.down")
+        if cfg.side_dim:
+            lw["side_gate"], lw["side_proj"], lw["side_norm"] = (get(pre + "side." + n) for n in ("gate", "proj", "norm"))
+        layers.append(lw)
+    return {"embed": get("embed"), "side_embed": get("side.embed") if cfg.side_dim else None,
+            "final_norm": get("final.norm"), "layers": layers}

@@ -35,19 +35,17 @@ import torch
 BLOCK_SIZE = 16
 
 
-class PagedKVCache:
-    def __init__(self, num_blocks: int, num_layers: int, num_kv_heads: int, head_dim: int,
-                 max_batch: int, max_blocks_per_seq: int, device="cuda", dtype=torch.float16,
+class BlockManager:
+    """Bookkeeping of the paged caches: blocks, request tables, table rows, prefix sharing and window eviction.
+    The pools themselves belong to the subclasses."""
+
+    def __init__(self, num_blocks: int, max_batch: int, max_blocks_per_seq: int, device="cuda",
                  enable_prefix_cache: bool = True, sliding_window: int = 0):
-        if num_blocks <= 0 or num_layers <= 0 or max_batch <= 0 or max_blocks_per_seq <= 0:
-            raise ValueError("num_blocks, num_layers, max_batch and max_blocks_per_seq must be positive")
-        self.num_blocks, self.num_layers = num_blocks, num_layers
-        self.num_kv_heads, self.head_dim = num_kv_heads, head_dim
+        if num_blocks <= 0 or max_batch <= 0 or max_blocks_per_seq <= 0:
+            raise ValueError("num_blocks, max_batch and max_blocks_per_seq must be positive")
+        self.num_blocks = num_blocks
         self.max_batch, self.max_blocks_per_seq = max_batch, max_blocks_per_seq
         self.device = torch.device(device)
-        shape = (num_blocks, num_kv_heads, BLOCK_SIZE, head_dim)
-        self.k_pools = [torch.zeros(shape, dtype=dtype, device=self.device) for _ in range(num_layers)]
-        self.v_pools = [torch.zeros(shape, dtype=dtype, device=self.device) for _ in range(num_layers)]
         # LIFO free list: the most recently freed block is reused first (manager.py:207, :260-275)
         self._free: List[int] = list(range(num_blocks - 1, -1, -1))
         self._tables: Dict[str, List[int]] = {}
@@ -261,6 +259,25 @@ class PagedKVCache:
             return self.block_table[: len(rows)], lens
         return self.block_table[self.batch_rows(request_ids)].contiguous(), lens
 
+    def check_errors(self) -> None:
+        """Raise if a kernel that worked on this cache recorded an error (subclasses with a status word)."""
+
+
+class PagedKVCache(BlockManager):
+    """K and V pools `[num_blocks, H_KV, 16, D]` per layer."""
+
+    def __init__(self, num_blocks: int, num_layers: int, num_kv_heads: int, head_dim: int,
+                 max_batch: int, max_blocks_per_seq: int, device="cuda", dtype=torch.float16,
+                 enable_prefix_cache: bool = True, sliding_window: int = 0):
+        if num_layers <= 0:
+            raise ValueError("num_layers must be positive")
+        super().__init__(num_blocks, max_batch, max_blocks_per_seq, device, enable_prefix_cache, sliding_window)
+        self.num_layers = num_layers
+        self.num_kv_heads, self.head_dim = num_kv_heads, head_dim
+        shape = (num_blocks, num_kv_heads, BLOCK_SIZE, head_dim)
+        self.k_pools = [torch.zeros(shape, dtype=dtype, device=self.device) for _ in range(num_layers)]
+        self.v_pools = [torch.zeros(shape, dtype=dtype, device=self.device) for _ in range(num_layers)]
+
     # ---- data path ----------------------------------------------------------------
     def append_decode(self, layer: int, request_ids: Sequence[str], q, k, v, cos, sin):
         """One decode step for one layer: rotate q / k and store k, v of each request's new token at
@@ -277,3 +294,41 @@ class PagedKVCache:
         table, lens = self.batch_view(request_ids)
         return ops.rope_append_paged_fp16(q, k, v, cos, sin, self.k_pools[layer], self.v_pools[layer], table, lens,
                                           self.max_blocks_per_seq, cu_seqlens=cu_seqlens, return_k=True)
+
+
+class HybridCache(BlockManager):
+    """What the layer runs of a hybrid decoder keep per request, behind one block table.
+
+    `specs` has one entry per layer run:
+      ("latent", row)            a pool [num_blocks, 16, stride] of cached rows of `row` elements (stride: row rounded up
+                                 to 16 bytes), addressed by the request's block table;
+      ("state", heads, dk, dv)   a recurrent state [max_batch, heads, dk, dv] in fp32, one slot per request, addressed
+                                 by the request's table row.  A slot is not cleared when it changes hands: a request's
+                                 state starts at zero because the kernels take the state of position 0 as zero.
+    The pages of a prefix do not bring back the recurrent state at its end, so prefixes are shared only by models
+    without one."""
+
+    def __init__(self, specs, num_blocks: int, max_batch: int, max_blocks_per_seq: int, device="cuda",
+                 dtype=torch.bfloat16):
+        super().__init__(num_blocks, max_batch, max_blocks_per_seq, device,
+                         enable_prefix_cache=all(s[0] == "latent" for s in specs))
+        self.dtype = dtype
+        align = 16 // torch.empty((), dtype=dtype).element_size()
+        self.stores = []
+        for spec in specs:
+            if spec[0] == "latent":
+                stride = (spec[1] + align - 1) // align * align
+                self.stores.append(torch.zeros((num_blocks, BLOCK_SIZE, stride), dtype=dtype, device=self.device))
+            elif spec[0] == "state":
+                self.stores.append(torch.zeros((max_batch,) + tuple(spec[1:]), dtype=torch.float32, device=self.device))
+            else:
+                raise ValueError(f"unknown store {spec[0]!r}")
+        self.status = torch.zeros(1, dtype=torch.int32, device=self.device)     # written by the kernels
+
+    def check_errors(self) -> None:
+        st = int(self.status.item())
+        if st:
+            self.status.zero_()
+            what = [text for bit, text in ((1, "a bounded wait ran out"),
+                                           (2, "a block-table entry or state slot outside the cache was met")) if st & bit]
+            raise RuntimeError("hybrid decoder kernels: " + "; ".join(what))

@@ -1,0 +1,74 @@
+/* C ABI of the hybrid decoder's operators (libfa_b200_hybrid.so, sm_100a): decayed linear attention, attention over
+ * cached latent rows, and the row-wise operators between the matrix products.
+ *
+ * Conventions: device pointers on the current device; every call is asynchronous on `stream` (a cudaStream_t);
+ * nothing is allocated.  `dtype` is the type of activations, weights and cached latent rows: FAH_F32 or FAH_BF16; the
+ * residual stream and the linear-attention state are always fp32.  `status` is one int32 in device memory that the
+ * caller has set to zero: a kernel that meets a block-table entry or a state slot outside the cache sets bit 1 in it
+ * and skips the access; a bounded wait that ran out sets bit 0.  Return value: 0, or a negative code with a text in
+ * fah_last_error(). */
+#ifndef FA_B200_HYBRID_H
+#define FA_B200_HYBRID_H
+#include <stddef.h>
+#include <stdint.h>
+
+#ifdef __cplusplus
+extern "C" {
+#endif
+
+enum { FAH_F32 = 0, FAH_BF16 = 1 };
+enum { FAH_OK = 0, FAH_ERR_INVALID_ARGUMENT = -1, FAH_ERR_UNSUPPORTED = -2, FAH_ERR_CUDA = -4 };
+
+const char* fah_last_error(void);
+
+/* x [rows, cols] fp32: embed_mode 1 adds embed[token], 2 sets x to embed[token]; then delta [rows, cols] is added, RMS-normed
+ * with weight delta_w first if that is given.  out [rows, cols] = rmsnorm(x) * w, or x itself if w is null; out may be null. */
+int fah_residual_norm(float* x, const void* delta, const void* delta_w, const void* embed, const int64_t* tokens,
+                      int embed_mode, int vocab, const void* w, void* out, int64_t rows, int cols, float eps, int dtype,
+                      void* stream);
+
+/* out [rows, cols] = rmsnorm(o [rows, cols]) * w * sigmoid(g), g with row stride g_stride. */
+int fah_gated_norm(const void* o, const void* g, int64_t g_stride, const void* w, void* out, int64_t rows, int cols, float eps,
+                   int dtype, void* stream);
+
+/* gu [rows, 2n]: out [rows, n] = g * sigmoid(alpha * g) * (u + shift), g = min(gu[:n], limit), u = clamp(gu[n:], -limit, limit). */
+int fah_clamped_glu(const void* gu, void* out, int64_t rows, int n, float limit, float alpha, float shift, int dtype,
+                    void* stream);
+
+/* out [rows, n] = gelu_tanh(z [rows, n]) * side[token, off : off + n], side with row stride side_stride. */
+int fah_side_gate(const void* z, const void* side, const int64_t* tokens, int vocab, int64_t side_stride, int off, void* out,
+                  int64_t rows, int n, int dtype, void* stream);
+
+/* Decayed linear attention with SiLU on q, k, v: per head S = decay * S + k v^T, o = S^T q.
+ * qkv [tokens, stride] with the heads x dk queries at column off_q, keys at off_k, heads x dv values at off_v;
+ * state [n_slots, heads, dk, dv] fp32; out [tokens, heads * dv].  cu_seqlens null: one token per sequence. */
+int fah_lightning(const void* qkv, int64_t stride, int off_q, int off_k, int off_v, int heads, int dk, int dv, const float* decay,
+                  float* state, int n_slots, const int32_t* slots, const int32_t* starts, const int32_t* cu_seqlens, int n_seq,
+                  int64_t tokens, void* out, int32_t* status, int dtype, void* stream);
+
+/* down [rows, down_stride]: the query latent at off_q, the key/value latent at off_kv and the shared key part at off_r.
+ * cq [rows, q_rank] and the latent c are RMS-normed, the shared part is rotated with cos / sin [rows, rot_dim / 2]; (c, rotated
+ * part) go to the row's place in pool [n_blocks, 16, pool_stride] and, where given, to c_out [rows, kv_rank] and
+ * r_out [rows, rot_dim]. */
+int fah_latent_prep(const void* down, int64_t down_stride, int off_q, int q_rank, int off_kv, int kv_rank, int off_r, int rot_dim,
+                    const void* wq, const void* wkv, float eps, const float* cos_t, const float* sin_t, void* cq, void* c_out,
+                    void* r_out, void* pool, int pool_stride, int n_blocks, const int32_t* block_table, int max_blocks, int n_seq,
+                    const int32_t* tok_seq, const int32_t* positions, int64_t rows, int32_t* status, int dtype, void* stream);
+
+/* Rotates columns [off, off + rot_dim) of every head of q [rows, heads * head_stride] in place (column i pairs with
+ * i + rot_dim / 2). */
+int fah_rotate_heads(void* q, const float* cos_t, const float* sin_t, int64_t rows, int heads, int head_stride, int off,
+                     int rot_dim, int dtype, void* stream);
+
+/* Attention over cached latent rows: every row of (q_abs [rows, heads, kv_rank] | rotated columns
+ * [q_off, q_off + rot_dim) of q [rows, heads, q_stride]) sees the keys 0 .. positions[row] of its sequence; values are the
+ * latents; the result times sigmoid(gate[row, head]) (gate may be null) goes to out [rows, heads, kv_rank]. */
+int fah_latent_attention(const void* q_abs, const void* q, int q_stride, int q_off, const float* cos_t, const float* sin_t,
+                         const void* pool, int pool_stride, int n_blocks, const int32_t* block_table, int max_blocks, int n_seq,
+                         const int32_t* tok_seq, const int32_t* positions, const void* gate, int64_t gate_stride, int heads,
+                         int kv_rank, int rot_dim, float scale, void* out, int64_t rows, int32_t* status, int dtype, void* stream);
+
+#ifdef __cplusplus
+}
+#endif
+#endif
