@@ -72,6 +72,9 @@ HYBRID_SIGNATURES = {
     "fah_rotate_heads": (_i, [_vp, _vp, _vp, _i64, _i, _i, _i, _i, _i, _vp]),
     "fah_latent_attention": (_i, [_vp, _vp, _i, _i, _vp, _vp, _vp, _i, _i, _vp, _i, _i, _vp, _vp, _vp, _i64, _i, _i, _i, _f, _vp,
                                   _i64, _vp, _i, _vp]),
+    "fah_latent_prefill": (_i, [_vp, _vp, _vp, _vp, _i64, _vp, _vp, _i, _i, _i64, _i64, _i, _i, _i, _i, _f, _vp, _vp, _vp]),
+    "fah_latent_prefill_supported": (_i, [_i, _i, _i, _f, _i]),
+    "fah_latent_gather": (_i, [_vp, _i, _i, _vp, _i, _i, _vp, _i64, _i, _i, _vp, _vp, _vp, _i, _vp]),
 }
 
 _lib = None

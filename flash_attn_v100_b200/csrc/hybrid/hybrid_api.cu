@@ -7,6 +7,7 @@
 
 #include "hybrid_common.cuh"
 #include "latent_attention.cuh"
+#include "latent_prefill.cuh"
 #include "lightning.cuh"
 #include "row_ops.cuh"
 
@@ -40,6 +41,16 @@ int sm_count() {
   if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return n;
   if (cached[dev] == 0 && cudaDeviceGetAttribute(&n, cudaDevAttrMultiProcessorCount, dev) == cudaSuccess) cached[dev] = n;
   return cached[dev] ? cached[dev] : n;
+}
+// cuTensorMapEncodeTiled, or null if the driver does not have it.
+void* tensor_map_encode() {
+  static void* fn = [] {
+    void* sym = nullptr;
+    cudaDriverEntryPointQueryResult qres;
+    const cudaError_t e = cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &sym, cudaEnableDefault, &qres);
+    return e == cudaSuccess && qres == cudaDriverEntryPointSuccess ? sym : nullptr;
+  }();
+  return fn;
 }
 constexpr int64_t kMaxRows = 1ll << 31;
 
@@ -151,6 +162,39 @@ int fah_latent_attention(const void* q_abs, const void* q, int q_stride, int q_o
   a.gate = gate; a.gate_stride = gate_stride; a.heads = heads; a.kv_rank = kv_rank; a.rot_dim = rot_dim; a.scale = scale; a.out = out; a.rows = rows;
   a.status = status;
   return done(FAH_DISPATCH(dtype, fa::hybrid::launch_latent_attention, a, st(stream)), "latent_attention");
+}
+
+int fah_latent_prefill_supported(int dim, int rot_dim, int vdim, float scale, int dtype) {
+  return dtype == FAH_BF16 && fa::hybrid::latent_prefill_supported(dim, rot_dim, vdim, scale) ? 1 : 0;
+}
+
+int fah_latent_prefill(const void* q, const void* kv, const void* kr, const void* gate, int64_t gate_stride, const int32_t* cu_q,
+                       const int32_t* cu_kv, int n_seq, int max_q, int64_t total_q, int64_t total_kv, int heads, int dim, int rot_dim, int vdim,
+                       float scale, void* out, int32_t* status, void* stream) {
+  FAH_REQUIRE(q && kv && kr && cu_q && cu_kv && out && status, "null pointer");
+  if (!fa::hybrid::latent_prefill_supported(dim, rot_dim, vdim, scale))
+    return fail(FAH_ERR_UNSUPPORTED, "latent_prefill is not built for dim=%d rot_dim=%d vdim=%d scale=%g", dim, rot_dim, vdim, (double)scale);
+  FAH_REQUIRE(heads > 0 && n_seq > 0 && max_q > 0 && total_q >= 0 && total_q < kMaxRows && total_kv >= total_q && total_kv < kMaxRows,
+              "bad sizes: heads=%d n_seq=%d max_q=%d total_q=%lld total_kv=%lld", heads, n_seq, max_q, (long long)total_q, (long long)total_kv);
+  FAH_REQUIRE(gate == nullptr || gate_stride >= heads, "gate_stride=%lld is smaller than heads=%d", (long long)gate_stride, heads);
+  for (const void* p : {q, kv, kr, (const void*)out})
+    FAH_REQUIRE((reinterpret_cast<uintptr_t>(p) & 15) == 0, "q, kv, kr and out must be 16-byte aligned");
+  void* enc = tensor_map_encode();
+  if (enc == nullptr) return fail(FAH_ERR_CUDA, "cuTensorMapEncodeTiled is not available from the driver");
+  fa::hybrid::LatentPrefillArgs a{q, kv, kr, gate, gate_stride, cu_q, cu_kv, n_seq, max_q, total_q, total_kv, heads, dim, rot_dim, vdim, scale, out,
+                                  status};
+  return done(fa::hybrid::launch_latent_prefill(a, enc, st(stream)), "latent_prefill");
+}
+
+int fah_latent_gather(const void* pool, int pool_stride, int n_blocks, const int32_t* block_table, int max_blocks, int n_seq, const int32_t* cu_kv,
+                      int64_t total_kv, int kv_rank, int rot_dim, void* c, void* r, int32_t* status, int dtype, void* stream) {
+  FAH_REQUIRE(dtype_ok(dtype), "unknown dtype %d", dtype);
+  FAH_REQUIRE(pool && block_table && cu_kv && c && r && status, "null pointer");
+  FAH_REQUIRE(kv_rank > 0 && rot_dim > 0 && pool_stride >= kv_rank + rot_dim && n_blocks > 0 && max_blocks > 0 && n_seq > 0 && total_kv >= 0 &&
+                  total_kv < kMaxRows,
+              "bad sizes: kv_rank=%d rot_dim=%d n_seq=%d total_kv=%lld", kv_rank, rot_dim, n_seq, (long long)total_kv);
+  fa::hybrid::LatentGatherArgs a{pool, pool_stride, n_blocks, block_table, max_blocks, n_seq, cu_kv, total_kv, kv_rank, rot_dim, c, r, status};
+  return done(FAH_DISPATCH(dtype, fa::hybrid::launch_latent_gather, a, st(stream)), "latent_gather");
 }
 
 }  // extern "C"

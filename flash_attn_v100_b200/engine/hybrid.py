@@ -11,6 +11,7 @@ between calls is described by `store` and lives in `HybridCache.stores`, one ent
 """
 from __future__ import annotations
 
+import itertools
 from dataclasses import dataclass
 from typing import List, Optional
 
@@ -36,6 +37,7 @@ class Step:
     block_table: torch.Tensor            # [n_seq, max_blocks] int32
     lens: Optional[List[int]]            # host: new tokens per sequence (None: one each)
     past: Optional[List[int]]            # host: cached tokens per sequence (prompts only)
+    cu_kv: Optional[torch.Tensor]        # [n_seq + 1] int32 offsets of all the sequences' keys (prompts only)
     status: torch.Tensor
 
 
@@ -68,8 +70,13 @@ class LightningMixer:
 class LatentAttentionMixer:
     """Attention on cached latent rows; keeps `kv_rank` + `rot_dim` elements per token."""
 
+    # Prompts of at least this many tokens per sequence expand the latents into per-head keys and values; shorter portions
+    # and decode steps work in the latent space, where nothing has to be computed for the keys.
+    EXPAND_TOKENS = 32
+
     def __init__(self, spec: LatentAttentionSpec, w: dict, eps: float):
         self.spec, self.w, self.eps = spec, w, eps
+        self.can_expand = w["w_in"].is_cuda and hops.latent_prefill_supported(spec.dim, spec.rot_dim, spec.vdim, spec.scale, w["w_in"].dtype)
 
     @staticmethod
     def store(spec: LatentAttentionSpec):
@@ -85,9 +92,19 @@ class LatentAttentionMixer:
         z = linear(h, w["w_in"])                                     # query latent | latent | shared key part | head gates
         at = w["in_at"]
         gate = z[:, at[3]:at[3] + H]
-        cq, _, _ = hops.latent_prep(z, at[0], s.q_rank, at[1], s.kv_rank, at[2], s.rot_dim, w["q_norm"], w["kv_norm"], self.eps, cos, sin,
-                                    store, step.block_table, step.tok_seq, step.positions, step.status)
-        q = linear(cq, w["w_uq"]).view(T, H, s.dim + s.rot_dim)
+        expand = self.can_expand and step.cu is not None and T >= self.EXPAND_TOKENS * len(step.lens)
+        fresh = expand and not any(step.past)
+        cq, c, kr = hops.latent_prep(z, at[0], s.q_rank, at[1], s.kv_rank, at[2], s.rot_dim, w["q_norm"], w["kv_norm"], self.eps, cos, sin,
+                                     store, step.block_table, step.tok_seq, step.positions, step.status, contiguous_kv=fresh)
+        q = linear(cq, w["w_uq"])
+        if expand:
+            if not fresh:                                            # this pass's rows are in the pages too
+                c, kr = hops.latent_gather(store, step.block_table, step.cu_kv, sum(step.past) + T, s.kv_rank, s.rot_dim, step.status)
+            hops.rotate_heads_(q, cos, sin, H, s.dim + s.rot_dim, s.dim, s.rot_dim)
+            o = hops.latent_prefill(q, linear(c, w["w_ukv"]), kr, gate, step.cu, step.cu_kv, max(step.lens), H, s.dim, s.vdim, s.scale,
+                                    step.status)
+            return linear(o, w["w_out"])
+        q = q.view(T, H, s.dim + s.rot_dim)
         # scores and values in the latent space: q W_uk against the cached latents, the weighted latent times W_uv
         q_abs = torch.empty((T, H, s.kv_rank), dtype=h.dtype, device=h.device)
         torch.bmm(q[..., :s.dim].transpose(0, 1), w["w_uk"], out=q_abs.transpose(0, 1))
@@ -170,7 +187,10 @@ class HybridDecoder(GreedyHead):
                                               torch.tensor(lens)).to(self.device, non_blocking=True)
         else:
             tok_seq = self._range(n_seq)
-        step = Step(token_ids, positions, slots, cu_seqlens, tok_seq, rows, block_table, lens, past, kv.status)
+        cu_kv = cu_seqlens
+        if prompt and any(past):
+            cu_kv = torch.tensor(list(itertools.accumulate((p + n for p, n in zip(past, lens)), initial=0)), dtype=torch.int32).to(self.device)
+        step = Step(token_ids, positions, slots, cu_seqlens, tok_seq, rows, block_table, lens, past, cu_kv, kv.status)
         if prompt and want is None:
             want = (cu_seqlens[1:] - 1).long()
         out = {}

@@ -197,3 +197,47 @@ def latent_attention(q_abs, q, q_off, cos, sin, pool, block_table, tok_seq, posi
         block_table.size(0), _p(tok_seq), _p(positions), _p(gate), gate.stride(0) if gate is not None else 0, heads, kv_rank, rot_dim, scale,
         _p(out), rows, _p(status), _DTYPE[T], _stream(q_abs)))
     return out
+
+
+def latent_prefill_supported(dim, rot_dim, vdim, scale, dtype):
+    """Whether `latent_prefill` is built for these sizes."""
+    return dtype in _DTYPE and bool(_lib.load_hybrid().fah_latent_prefill_supported(dim, rot_dim, vdim, scale, _DTYPE[dtype]))
+
+
+def latent_prefill(q, kv, kr, gate, cu_q, cu_kv, max_q, heads, dim, vdim, scale, status):
+    """Causal prompt attention on expanded latents (bfloat16): q [total_q, heads * (dim + rot_dim)] rotated, kv [total_kv,
+    heads * (dim + vdim)] = keys | values, kr [total_kv, rot_dim].  A sequence's queries are its last keys.
+    Returns [total_q, heads * vdim], head h times sigmoid(gate[:, h])."""
+    T = torch.bfloat16
+    for name, t in (("q", q), ("kv", kv), ("kr", kr)):
+        _check(t, name, T)
+    for name, t in (("cu_q", cu_q), ("cu_kv", cu_kv), ("status", status)):
+        _check(t, name, torch.int32)
+    rot_dim = kr.size(1)
+    if q.size(1) != heads * (dim + rot_dim) or kv.shape != (kr.size(0), heads * (dim + vdim)) or cu_q.numel() != cu_kv.numel():
+        raise RuntimeError("q, kv and kr do not fit the head sizes")
+    if gate is not None:
+        _check(gate, "gate", T, contiguous=False)
+        if gate.shape != (q.size(0), heads) or gate.stride(1) != 1:
+            raise RuntimeError("gate must be [total_q, heads] with contiguous rows")
+    out = torch.empty((q.size(0), heads * vdim), dtype=T, device=q.device)
+    _lib.check_hybrid(_lib.load_hybrid().fah_latent_prefill(
+        _p(q), _p(kv), _p(kr), _p(gate), gate.stride(0) if gate is not None else 0, _p(cu_q), _p(cu_kv), cu_q.numel() - 1, max_q, q.size(0),
+        kv.size(0), heads, dim, rot_dim, vdim, scale, _p(out), _p(status), _stream(q)))
+    return out
+
+
+def latent_gather(pool, block_table, cu_kv, total_kv, kv_rank, rot_dim, status):
+    """The cached latent rows of every sequence as contiguous rows: ([total_kv, kv_rank], [total_kv, rot_dim])."""
+    T = _type(pool, "pool")
+    _check(pool, "pool", T)
+    for name, t in (("cu_kv", cu_kv), ("status", status), ("block_table", block_table)):
+        _check(t, name, torch.int32)
+    if block_table.size(0) != cu_kv.numel() - 1:
+        raise RuntimeError("cu_kv must have one entry more than block_table has rows")
+    c = torch.empty((total_kv, kv_rank), dtype=T, device=pool.device)
+    r = torch.empty((total_kv, rot_dim), dtype=T, device=pool.device)
+    _lib.check_hybrid(_lib.load_hybrid().fah_latent_gather(
+        _p(pool), pool.size(2), pool.size(0), _p(block_table), block_table.size(1), block_table.size(0), _p(cu_kv), total_kv, kv_rank, rot_dim,
+        _p(c), _p(r), _p(status), _DTYPE[T], _stream(pool)))
+    return c, r

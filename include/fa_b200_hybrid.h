@@ -68,6 +68,19 @@ int fah_latent_attention(const void* q_abs, const void* q, int q_stride, int q_o
                          const int32_t* tok_seq, const int32_t* positions, const void* gate, int64_t gate_stride, int heads,
                          int kv_rank, int rot_dim, float scale, void* out, int64_t rows, int32_t* status, int dtype, void* stream);
 
+/* Prompt attention on expanded latents (bfloat16): q [total_q, heads, dim + rot_dim] rotated, kv [total_kv, heads * dim | heads *
+ * vdim], kr [total_kv, rot_dim] shared by the heads.  A sequence's queries are its last keys; causal.  The result times
+ * sigmoid(gate[row, head]) (gate may be null) goes to out [total_q, heads * vdim].  Sizes: fah_latent_prefill_supported. */
+int fah_latent_prefill(const void* q, const void* kv, const void* kr, const void* gate, int64_t gate_stride, const int32_t* cu_q,
+                       const int32_t* cu_kv, int n_seq, int max_q, int64_t total_q, int64_t total_kv, int heads, int dim, int rot_dim,
+                       int vdim, float scale, void* out, int32_t* status, void* stream);
+int fah_latent_prefill_supported(int dim, int rot_dim, int vdim, float scale, int dtype);
+
+/* Cached latent rows of every sequence as contiguous rows: c [total_kv, kv_rank], r [total_kv, rot_dim]. */
+int fah_latent_gather(const void* pool, int pool_stride, int n_blocks, const int32_t* block_table, int max_blocks, int n_seq,
+                      const int32_t* cu_kv, int64_t total_kv, int kv_rank, int rot_dim, void* c, void* r, int32_t* status, int dtype,
+                      void* stream);
+
 #ifdef __cplusplus
 }
 #endif
