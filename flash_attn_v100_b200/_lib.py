@@ -67,11 +67,13 @@ HYBRID_SIGNATURES = {
     "fah_gated_norm": (_i, [_vp, _vp, _i64, _vp, _vp, _i64, _i, _f, _i, _vp]),
     "fah_clamped_glu": (_i, [_vp, _vp, _i64, _i, _f, _f, _f, _i, _vp]),
     "fah_side_gate": (_i, [_vp, _vp, _vp, _i, _i64, _i, _vp, _i64, _i, _i, _vp]),
-    "fah_lightning": (_i, [_vp, _i64] + [_i] * 6 + [_vp, _vp, _i, _vp, _vp, _vp, _i, _i64, _vp, _vp, _i, _vp]),
+    "fah_lightning_workspace": (_sz, [_i] * 6),
+    "fah_lightning": (_i, [_vp, _i64] + [_i] * 6 + [_vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i64, _vp, _vp, _sz, _vp, _i, _vp]),
     "fah_latent_prep": (_i, [_vp, _i64] + [_i] * 6 + [_vp, _vp, _f] + [_vp] * 6 + [_i, _i, _vp, _i, _i, _vp, _vp, _i64, _vp, _i, _vp]),
     "fah_rotate_heads": (_i, [_vp, _vp, _vp, _i64, _i, _i, _i, _i, _i, _vp]),
+    "fah_latent_attention_workspace": (_sz, [_i, _i, _i, _i64, _i]),
     "fah_latent_attention": (_i, [_vp, _vp, _i, _i, _vp, _vp, _vp, _i, _i, _vp, _i, _i, _vp, _vp, _vp, _i64, _i, _i, _i, _f, _vp,
-                                  _i64, _vp, _i, _vp]),
+                                  _i64, _vp, _sz, _vp, _i, _vp]),
     "fah_latent_prefill": (_i, [_vp, _vp, _vp, _vp, _i64, _vp, _vp, _i, _i, _i64, _i64, _i, _i, _i, _i, _f, _vp, _vp, _vp]),
     "fah_latent_prefill_supported": (_i, [_i, _i, _i, _f, _i]),
     "fah_latent_gather": (_i, [_vp, _i, _i, _vp, _i, _i, _vp, _i64, _i, _i, _vp, _vp, _vp, _i, _vp]),

@@ -100,9 +100,16 @@ int fah_side_gate(const void* z, const void* side, const int64_t* tokens, int vo
   return done(FAH_DISPATCH(dtype, fa::hybrid::launch_side_gate, z, side, tokens, vocab, side_stride, off, out, rows, n, st(stream)), "side_gate");
 }
 
+size_t fah_lightning_workspace(int n_seq, int heads, int dk, int dv, int max_len, int dtype) {
+  if (dtype != FAH_BF16 || n_seq <= 0 || heads <= 0 || dk <= 0 || dv <= 0 || max_len <= 0) return 0;
+  int seg_len = 0;
+  const int segs = fa::hybrid::lightning_segments(n_seq, heads, dv, max_len, sm_count(), &seg_len);
+  return segs > 1 ? (size_t)n_seq * segs * heads * dk * dv * sizeof(float) : 0;
+}
+
 int fah_lightning(const void* qkv, int64_t stride, int off_q, int off_k, int off_v, int heads, int dk, int dv, const float* decay, float* state,
-                  int n_slots, const int32_t* slots, const int32_t* starts, const int32_t* cu_seqlens, int n_seq, int64_t tokens, void* out,
-                  int32_t* status, int dtype, void* stream) {
+                  int n_slots, const int32_t* slots, const int32_t* starts, const int32_t* cu_seqlens, int n_seq, int max_len, int64_t tokens,
+                  void* out, void* workspace, size_t workspace_bytes, int32_t* status, int dtype, void* stream) {
   FAH_REQUIRE(dtype_ok(dtype), "unknown dtype %d", dtype);
   FAH_REQUIRE(qkv && decay && state && slots && starts && out && status, "null pointer");
   FAH_REQUIRE(heads > 0 && heads < 65536 && dk > 0 && dv > 0 && n_slots > 0, "bad sizes: heads=%d dk=%d dv=%d slots=%d", heads, dk, dv, n_slots);
@@ -118,6 +125,15 @@ int fah_lightning(const void* qkv, int64_t stride, int off_q, int off_k, int off
   a.cu = cu_seqlens; a.n_seq = n_seq; a.total = tokens; a.out = out; a.status = status;
   if (fa::hybrid::lightning_decode_supported(a))
     return done(FAH_DISPATCH(dtype, fa::hybrid::launch_lightning_decode, a, sm_count(), st(stream)), "lightning_decode");
+  if (dtype == FAH_BF16 && fa::hybrid::lightning_chunk_supported(a)) {
+    FAH_REQUIRE(max_len > 0, "prompts need max_len");
+    const size_t need = fah_lightning_workspace(n_seq, heads, dk, dv, max_len, dtype);
+    FAH_REQUIRE(workspace_bytes >= need && (need == 0 || (workspace != nullptr && (reinterpret_cast<uintptr_t>(workspace) & 15) == 0)),
+                "the workspace has %zu bytes, %zu (16-byte aligned) are needed", workspace_bytes, need);
+    a.max_segs = fa::hybrid::lightning_segments(n_seq, heads, dv, max_len, sm_count(), &a.seg_len);
+    a.seg_state = static_cast<float*>(workspace);
+    return done(fa::hybrid::launch_lightning_chunk(a, st(stream)), "lightning_chunk");
+  }
   return done(FAH_DISPATCH(dtype, fa::hybrid::launch_lightning_scan, a, st(stream)), "lightning_scan");
 }
 
@@ -146,10 +162,16 @@ int fah_rotate_heads(void* q, const float* cos_t, const float* sin_t, int64_t ro
   return done(FAH_DISPATCH(dtype, fa::hybrid::launch_rotate_heads, q, cos_t, sin_t, rows, heads, head_stride, off, rot_dim, st(stream)), "rotate_heads");
 }
 
+size_t fah_latent_attention_workspace(int heads, int kv_rank, int rot_dim, int64_t rows, int dtype) {
+  if (dtype != FAH_BF16 || heads <= 0 || rows <= 0 || kv_rank <= 0) return 0;
+  const int64_t n = fa::hybrid::latent_decode_ctas(heads, sm_count());
+  return (size_t)(n * 2 * heads * ((int64_t)kv_rank + 2) * 4 + (rows + 1) * 4);
+}
+
 int fah_latent_attention(const void* q_abs, const void* q, int q_stride, int q_off, const float* cos_t, const float* sin_t, const void* pool,
                          int pool_stride, int n_blocks, const int32_t* block_table, int max_blocks, int n_seq, const int32_t* tok_seq,
                          const int32_t* positions, const void* gate, int64_t gate_stride, int heads, int kv_rank, int rot_dim, float scale, void* out,
-                         int64_t rows, int32_t* status, int dtype, void* stream) {
+                         int64_t rows, void* workspace, size_t workspace_bytes, int32_t* status, int dtype, void* stream) {
   FAH_REQUIRE(dtype_ok(dtype), "unknown dtype %d", dtype);
   FAH_REQUIRE(q_abs && q && cos_t && sin_t && pool && block_table && tok_seq && positions && out && status, "null pointer");
   FAH_REQUIRE(heads > 0 && heads < 65536 && kv_rank > 0 && kv_rank <= 16384 && rot_dim >= 0 && rot_dim % 2 == 0 && q_off >= 0 && q_off + rot_dim <= q_stride,
@@ -161,6 +183,16 @@ int fah_latent_attention(const void* q_abs, const void* q, int q_stride, int q_o
   a.n_blocks = n_blocks; a.block_table = block_table; a.max_blocks = max_blocks; a.n_seq = n_seq; a.tok_seq = tok_seq; a.positions = positions;
   a.gate = gate; a.gate_stride = gate_stride; a.heads = heads; a.kv_rank = kv_rank; a.rot_dim = rot_dim; a.scale = scale; a.out = out; a.rows = rows;
   a.status = status;
+  if (dtype == FAH_BF16 && fa::hybrid::latent_decode_supported(a)) {
+    const size_t need = fah_latent_attention_workspace(heads, kv_rank, rot_dim, rows, dtype);
+    FAH_REQUIRE(workspace_bytes >= need && (need == 0 || (workspace != nullptr && (reinterpret_cast<uintptr_t>(workspace) & 15) == 0)),
+                "the workspace has %zu bytes, %zu (16-byte aligned) are needed", workspace_bytes, need);
+    a.n_cta = fa::hybrid::latent_decode_ctas(heads, sm_count());
+    a.part_o = static_cast<float*>(workspace);
+    a.part_ml = a.part_o + (int64_t)a.n_cta * 2 * heads * kv_rank;
+    a.row_tiles = reinterpret_cast<int32_t*>(a.part_ml + (int64_t)a.n_cta * 2 * heads * 2);
+    return done(fa::hybrid::launch_latent_decode(a, st(stream)), "latent_decode");
+  }
   return done(FAH_DISPATCH(dtype, fa::hybrid::launch_latent_attention, a, st(stream)), "latent_attention");
 }
 

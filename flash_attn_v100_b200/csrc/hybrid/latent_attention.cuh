@@ -24,14 +24,21 @@ struct LatentAttentionArgs {
   void* out;                 // T [rows, heads, kv_rank]
   long long rows;
   int* status;
-  // split-KV decode only
-  int n_split;
-  float* part_o;             // [n_split, rows, heads, kv_rank]
-  float* part_ml;            // [n_split, rows, heads, 2] (maximum in log2 units, sum)
+  // tensor-core kernel: work is cut into equal runs of key tiles, one per CTA and head block
+  int n_cta;
+  float* part_o;             // [n_cta, 2, heads, kv_rank] unnormalised sums of the rows that are cut
+  float* part_ml;            // [n_cta, 2, heads, 2]: their maxima (log2 units) and weights
+  int32_t* row_tiles;        // [rows + 1] prefix sums of the rows' key tiles, written by the kernel for the merge
 };
 
 // One CTA per (row, head): any size, both types.
 template <typename T> cudaError_t launch_latent_attention(const LatentAttentionArgs& a, cudaStream_t s);
+
+
+// Tensor cores (bfloat16; kv_rank + rot_dim <= 576, both multiples of 8).
+bool latent_decode_supported(const LatentAttentionArgs& a);
+int latent_decode_ctas(int heads, int sm_count);   // per head block
+cudaError_t launch_latent_decode(const LatentAttentionArgs& a, cudaStream_t s);
 
 }  // namespace hybrid
 }  // namespace fa

@@ -1,0 +1,433 @@
+// Attention in the latent space on the tensor cores (mma.sync, bfloat16 operands, fp32 scores, weights' sums and
+// accumulators), sm_100a: decode steps and short portions of prompts.
+//
+// All heads read the same cached rows, so a key tile (64 tokens) is fetched once and serves every head of the block (16 or
+// 32, the M rows of the MMAs) as key and as value.  The (row, key tile) units of the batch are numbered row by row and cut
+// into equal runs, one per CTA, whatever the lengths; a row that is cut leaves partial sums that a second kernel merges.
+//
+// Eight warps.  Scores: warp = (half of the tile's keys) x (quarter of the columns); its quarter of Q stays in registers for
+// the whole row, and the four partial score tiles are added up in shared memory by the softmax.  Values: warp = an eighth of the
+// latent's columns.  The next tile is copied (cp.async) while the current one is computed.
+#include <math_constants.h>
+
+#include "../common.cuh"
+#include "hybrid_common.cuh"
+#include "latent_attention.cuh"
+
+namespace fa {
+namespace hybrid {
+namespace {
+
+constexpr int KT = 64;         // keys per tile
+constexpr int kThreads = 256;
+constexpr int kSPad = KT + 4;  // row stride of the partial score tiles
+
+// Unit (16 bytes) `u` of key row `row`, swizzled within groups of eight units.
+template <int UNITS>
+__device__ __forceinline__ uint32_t key_off(int row, int u) {
+  return (uint32_t)((row * UNITS + ((u & ~7) | ((u ^ row) & 7))) * 16);
+}
+
+__device__ __forceinline__ int row_tiles_of(const LatentAttentionArgs& a, long long row) {
+  const int n = a.positions[row] + 1;
+  return n > 0 ? (n + KT - 1) / KT : 1;
+}
+
+// Inclusive scan over the block of one int per thread; `buf` holds 8 ints.
+__device__ __forceinline__ int block_scan(int v, int* buf) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const int t = __shfl_up_sync(0xffffffffu, v, o);
+    if (lane >= o) v += t;
+  }
+  if (lane == 31) buf[warp] = v;
+  __syncthreads();
+  int add = 0;
+  for (int i = 0; i < warp; ++i) add += buf[i];
+  __syncthreads();
+  return v + add;
+}
+
+// KS: 16-column steps per warp quarter (4 * 16 * KS >= kv_rank + rot_dim); MB: 16-head blocks.
+template <int KS, int MB>
+__global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const LatentAttentionArgs a) {
+  constexpr int UNITS = KS * 8;                    // 16-byte units per key row
+  constexpr int STAGE = KT * UNITS * 16;
+  constexpr int M = 16 * MB;
+  constexpr int TPR = kThreads / M;                // softmax threads per row
+  constexpr int KPT = KT / TPR;                    // keys per softmax thread
+  extern __shared__ __align__(1024) uint8_t sm[];
+  const uint32_t sKV = smem_u32(sm);
+  float* sS = reinterpret_cast<float*>(sm + 2 * STAGE);            // [4][M][kSPad]
+  const uint32_t sP = smem_u32(sS + 4 * M * kSPad);                // [M][KT] bfloat16, swizzled
+  float* sAlpha = reinterpret_cast<float*>(sm + 2 * STAGE + 4 * M * kSPad * 4 + M * KT * 2);   // [M]
+  float* sL = sAlpha + M;                                          // [M]
+  int* scan_buf = reinterpret_cast<int*>(sL + M);                  // [8]
+  int* found = scan_buf + 8;                                       // [2] first row, its first unit
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+  const int cta = blockIdx.x, h0 = blockIdx.y * M;
+  const int R = a.kv_rank, D = R + a.rot_dim;
+
+  // ---- my run of units --------------------------------------------------------------------------
+  int total = 0;
+  for (long long r0 = 0; r0 < a.rows; r0 += kThreads) {
+    const int v = r0 + tid < a.rows ? row_tiles_of(a, r0 + tid) : 0;
+    const int inc = block_scan(v, scan_buf);
+    if (cta == 0 && blockIdx.y == 0 && r0 + tid < a.rows) a.row_tiles[r0 + tid + 1] = total + inc;
+    if (tid == kThreads - 1) found[0] = inc;
+    __syncthreads();
+    total += found[0];
+    __syncthreads();
+  }
+  if (cta == 0 && blockIdx.y == 0 && tid == 0) a.row_tiles[0] = 0;
+  const int per = (total + a.n_cta - 1) / a.n_cta;
+  const int u0 = cta * per, u1 = min(u0 + per, total);
+  if (u0 >= u1) return;
+  {
+    int base = 0;
+    for (long long r0 = 0; r0 < a.rows; r0 += kThreads) {
+      const int v = r0 + tid < a.rows ? row_tiles_of(a, r0 + tid) : 0;
+      const int inc = base + block_scan(v, scan_buf);
+      if (v > 0 && inc - v <= u0 && u0 < inc) { found[0] = (int)(r0 + tid); found[1] = inc - v; }
+      if (tid == kThreads - 1) scan_buf[0] = inc;
+      __syncthreads();
+      base = scan_buf[0];
+      __syncthreads();
+      if (base > u0) break;
+    }
+  }
+  const int first_row = found[0];
+  struct Cursor { int row, tile, tiles; };
+  auto start_row = [&](Cursor& c, int row) { c.row = row; c.tile = 0; c.tiles = row_tiles_of(a, row); };
+  auto advance = [&](Cursor& c) {
+    if (++c.tile == c.tiles && c.row + 1 < a.rows) start_row(c, c.row + 1);
+  };
+
+  // ---- copies -----------------------------------------------------------------------------------
+  bool bad = false;
+  // lane 0-3 of every warp: pages of the cursor's tile
+  auto tile_pages = [&](const Cursor& c) {
+    int page = -1;
+    const int seq = a.tok_seq[c.row], n = a.positions[c.row] + 1, key = c.tile * KT + lane * 16;
+    if (lane < 4 && key < n) {
+      if (seq >= 0 && seq < a.n_seq && (key >> 4) < a.max_blocks) page = a.block_table[(long long)seq * a.max_blocks + (key >> 4)];
+      if (page < 0 || page >= a.n_blocks) { page = -1; bad = true; }
+    }
+    return page;
+  };
+  auto copy_tile = [&](const Cursor& c, int page, int stage) {
+    const int n = a.positions[c.row] + 1 - c.tile * KT;     // keys of the tile that exist
+    const bf16* pool = static_cast<const bf16*>(a.pool);
+#pragma unroll
+    for (int i = 0; i < KT * UNITS / kThreads; ++i) {
+      const int idx = tid + i * kThreads, key = idx / UNITS, u = idx - key * UNITS;
+      // the page's owner lane differs within a warp only where a warp's units straddle two rows
+      const int pg = __shfl_sync(0xffffffffu, page, key >> 4);
+      const bool ok = pg >= 0 && key < n && u * 8 < a.pool_stride;
+      const bf16* src = pool + ((long long)(ok ? pg : 0) * 16 + (key & 15)) * a.pool_stride + (ok ? u * 8 : 0);
+      cp_async_16(sKV + stage * STAGE + key_off<UNITS>(key, u), src, ok);
+    }
+  };
+
+  // ---- per-row state ----------------------------------------------------------------------------
+  const int slice = warp & 3, khalf = warp >> 2;
+  uint32_t qf[MB][KS][4];
+  float o[MB][KS][4];
+  auto q_elem = [&](long long row, int head, int c) -> float {
+    if (head >= a.heads || c >= D) return 0.f;
+    if (c < R) return to_f(static_cast<const bf16*>(a.q_abs)[(row * a.heads + head) * R + c]);
+    const int half = a.rot_dim / 2, i = c - R, f = i < half ? i : i - half;
+    const bf16* qr = static_cast<const bf16*>(a.q) + (row * a.heads + head) * a.q_stride + a.q_off;
+    const float cs = a.cos_t[row * half + f], sn = a.sin_t[row * half + f];
+    return i < half ? to_f(qr[i]) * cs - to_f(qr[i + half]) * sn : to_f(qr[i]) * cs + to_f(qr[i - half]) * sn;
+  };
+  auto load_q = [&](long long row) {
+#pragma unroll
+    for (int m = 0; m < MB; ++m)
+#pragma unroll
+      for (int k = 0; k < KS; ++k)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int head = h0 + m * 16 + g + (e & 1) * 8, c = (slice * KS + k) * 16 + t4 * 2 + (e >> 1) * 8;
+          if (c + 1 < R && head < a.heads)         // two latent columns at once (kv_rank is a multiple of 8)
+            qf[m][k][e] = *reinterpret_cast<const uint32_t*>(static_cast<const bf16*>(a.q_abs) + (row * a.heads + head) * R + c);
+          else
+            qf[m][k][e] = pack_bf162(q_elem(row, head, c), q_elem(row, head, c + 1));
+        }
+#pragma unroll
+    for (int m = 0; m < MB; ++m)
+#pragma unroll
+      for (int n = 0; n < KS; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[m][n][e] = 0.f;
+  };
+  const int srow = tid / TPR, sk0 = (tid % TPR) * KPT;       // softmax: my head row and first key
+  float m_run = -CUDART_INF_F, l_run = 0.f;
+  const float sc = a.scale * 1.4426950408889634f;
+
+  Cursor cur;
+  start_row(cur, first_row);
+  cur.tile = u0 - found[1];
+  Cursor nxt = cur;
+  int piece_tile0 = cur.tile;
+  copy_tile(nxt, tile_pages(nxt), 0);
+  cp_async_commit();
+  int page_next = -1;
+  if (u0 + 1 < u1) {
+    advance(nxt);
+    page_next = tile_pages(nxt);
+  }
+  load_q(cur.row);
+
+  for (int u = u0; u < u1; ++u) {
+    const int stage = (u - u0) & 1;
+    cp_async_wait<0>();
+    __syncthreads();                                // tile u has landed; the other stage is no longer read
+    if (u + 1 < u1) {
+      copy_tile(nxt, page_next, stage ^ 1);
+      cp_async_commit();
+      if (u + 2 < u1) {
+        advance(nxt);
+        page_next = tile_pages(nxt);
+      }
+    }
+    // ---- partial scores -------------------------------------------------------------------------
+    {
+      float s[MB][4][4];
+#pragma unroll
+      for (int m = 0; m < MB; ++m)
+#pragma unroll
+        for (int n = 0; n < 4; ++n)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) s[m][n][e] = 0.f;
+#pragma unroll
+      for (int k = 0; k < KS; ++k) {
+#pragma unroll
+        for (int n2 = 0; n2 < 2; ++n2) {
+          uint32_t b[4];
+          const int key = khalf * 32 + n2 * 16 + (lane & 7) + (lane >> 4) * 8;
+          ldmatrix_x4(b, sKV + stage * STAGE + key_off<UNITS>(key, (slice * KS + k) * 2 + ((lane >> 3) & 1)));
+#pragma unroll
+          for (int m = 0; m < MB; ++m) {
+            mma_bf16_16816(s[m][n2 * 2], qf[m][k], b[0], b[1]);
+            mma_bf16_16816(s[m][n2 * 2 + 1], qf[m][k], b[2], b[3]);
+          }
+        }
+      }
+#pragma unroll
+      for (int m = 0; m < MB; ++m)
+#pragma unroll
+        for (int n = 0; n < 4; ++n)
+#pragma unroll
+          for (int h = 0; h < 2; ++h)
+            *reinterpret_cast<float2*>(sS + (slice * M + m * 16 + g + h * 8) * kSPad + khalf * 32 + n * 8 + t4 * 2) =
+                make_float2(s[m][n][2 * h], s[m][n][2 * h + 1]);
+    }
+    __syncthreads();
+    // ---- softmax of my row's keys ---------------------------------------------------------------
+    {
+      const int valid = a.positions[cur.row] + 1 - cur.tile * KT;
+      float p[KPT];
+      float mx = -CUDART_INF_F;
+#pragma unroll
+      for (int i = 0; i < KPT; i += 4) {
+        float4 v = *reinterpret_cast<const float4*>(sS + srow * kSPad + sk0 + i);
+#pragma unroll
+        for (int q = 1; q < 4; ++q) {
+          const float4 w = *reinterpret_cast<const float4*>(sS + (q * M + srow) * kSPad + sk0 + i);
+          v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w;
+        }
+        p[i] = v.x; p[i + 1] = v.y; p[i + 2] = v.z; p[i + 3] = v.w;
+      }
+#pragma unroll
+      for (int i = 0; i < KPT; ++i) {
+        p[i] = sk0 + i < valid ? p[i] * sc : -CUDART_INF_F;
+        mx = fmaxf(mx, p[i]);
+      }
+#pragma unroll
+      for (int w = 1; w < TPR; w <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, w));
+      const float m_new = fmaxf(m_run, mx);
+      const float ref = m_new == -CUDART_INF_F ? 0.f : m_new;
+      const float alpha = exp2f(m_run - ref);       // 0 at the row's first tile
+      float sum = 0.f;
+#pragma unroll
+      for (int i = 0; i < KPT; ++i) { p[i] = exp2f(p[i] - ref); sum += p[i]; }
+#pragma unroll
+      for (int w = 1; w < TPR; w <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, w);
+      l_run = l_run * alpha + sum;
+      m_run = m_new;
+#pragma unroll
+      for (int i = 0; i < KPT; i += 4) {
+        const int c = sk0 + i;
+        const uint32_t addr = sP + (uint32_t)((srow * 8 + ((c >> 3) ^ (srow & 7))) * 16 + (c & 7) * 2);
+        asm volatile("st.shared.v2.b32 [%0], {%1,%2};" ::"r"(addr), "r"(pack_bf162(p[i], p[i + 1])), "r"(pack_bf162(p[i + 2], p[i + 3]))
+                     : "memory");
+      }
+      if (tid % TPR == 0) { sAlpha[srow] = alpha; sL[srow] = l_run; }
+    }
+    __syncthreads();
+    // ---- values: my columns of the latents --------------------------------------------------------
+    {
+#pragma unroll
+      for (int m = 0; m < MB; ++m) {
+        const float a0 = sAlpha[m * 16 + g], a1 = sAlpha[m * 16 + g + 8];
+        if (__any_sync(0xffffffffu, a0 != 1.f || a1 != 1.f)) {
+#pragma unroll
+          for (int n = 0; n < KS; ++n) { o[m][n][0] *= a0; o[m][n][1] *= a0; o[m][n][2] *= a1; o[m][n][3] *= a1; }
+        }
+      }
+#pragma unroll
+      for (int k2 = 0; k2 < KT / 32; ++k2) {        // 32 keys at a time
+        uint32_t pf[MB][2][4];
+#pragma unroll
+        for (int m = 0; m < MB; ++m)
+#pragma unroll
+          for (int k = 0; k < 2; ++k) {
+            const int r = m * 16 + (lane & 15), c8 = (k2 * 2 + k) * 2 + (lane >> 4);
+            ldmatrix_x4(pf[m][k], sP + (uint32_t)((r * 8 + (c8 ^ (r & 7))) * 16));
+          }
+#pragma unroll
+        for (int n = 0; n < KS; ++n) {
+          if ((warp * KS + n) * 8 < R) {
+            uint32_t b[4];
+            ldmatrix_x4_trans(b, sKV + stage * STAGE + key_off<UNITS>(k2 * 32 + lane, warp * KS + n));
+#pragma unroll
+            for (int m = 0; m < MB; ++m) {
+              mma_bf16_16816(o[m][n], pf[m][0], b[0], b[1]);
+              mma_bf16_16816(o[m][n], pf[m][1], b[2], b[3]);
+            }
+          }
+        }
+      }
+    }
+    // ---- end of a row or of my run ------------------------------------------------------------------
+    const bool row_end = cur.tile + 1 == cur.tiles;
+    if (row_end || u + 1 == u1) {
+      const bool whole = row_end && piece_tile0 == 0;
+      const int which = cur.row == first_row ? 0 : 1;
+      if (!whole && tid % TPR == 0 && h0 + srow < a.heads) {
+        float* ml = a.part_ml + (((long long)cta * 2 + which) * a.heads + h0 + srow) * 2;
+        ml[0] = m_run;
+        ml[1] = l_run;
+      }
+#pragma unroll
+      for (int m = 0; m < MB; ++m)
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          const int head = h0 + m * 16 + g + h * 8;
+          if (head < a.heads) {
+            float f = 1.f;
+            if (whole) {
+              const float l = sL[m * 16 + g + h * 8];
+              f = l > 0.f ? 1.f / l : 0.f;
+              if (a.gate != nullptr) f *= sigmoid_f(to_f(static_cast<const bf16*>(a.gate)[(long long)cur.row * a.gate_stride + head]));
+            }
+#pragma unroll
+            for (int n = 0; n < KS; ++n) {
+              const int c = (warp * KS + n) * 8 + t4 * 2;
+              if (c < R) {
+                const float x = o[m][n][2 * h] * f, y = o[m][n][2 * h + 1] * f;
+                if (whole)
+                  *reinterpret_cast<uint32_t*>(static_cast<bf16*>(a.out) + ((long long)cur.row * a.heads + head) * R + c) = pack_bf162(x, y);
+                else
+                  *reinterpret_cast<float2*>(a.part_o + (((long long)cta * 2 + which) * a.heads + head) * R + c) = make_float2(x, y);
+              }
+            }
+          }
+        }
+      if (u + 1 < u1) {
+        m_run = -CUDART_INF_F;
+        l_run = 0.f;
+        load_q(cur.row + 1);
+        piece_tile0 = 0;
+      }
+    }
+    if (u + 1 < u1) advance(cur);
+  }
+  if (bad) atomicOr(a.status, 2);
+}
+
+// Rows that several CTAs worked on: log-sum-exp merge of their partial sums.  One CTA per (row, head).
+__global__ void __launch_bounds__(128) latent_decode_merge_kernel(const LatentAttentionArgs a) {
+  const long long row = blockIdx.x;
+  const int head = blockIdx.y;
+  const int b0 = a.row_tiles[row], b1 = a.row_tiles[row + 1], total = a.row_tiles[a.rows];
+  const int per = (total + a.n_cta - 1) / a.n_cta;
+  const int c0 = b0 / per, c1 = (b1 - 1) / per;
+  if (c0 == c1) return;                             // one CTA had the whole row
+  // the row is CTA c's first one exactly if the CTA's run starts inside it or at its first unit
+  float m = -CUDART_INF_F;
+  for (int c = c0; c <= c1; ++c) {
+    const int which = c * per >= b0 ? 0 : 1;
+    m = fmaxf(m, a.part_ml[(((long long)c * 2 + which) * a.heads + head) * 2]);
+  }
+  float l = 0.f;
+  for (int c = c0; c <= c1; ++c) {
+    const float* ml = a.part_ml + (((long long)c * 2 + (c * per >= b0 ? 0 : 1)) * a.heads + head) * 2;
+    l += ml[1] * exp2f(ml[0] - m);
+  }
+  float f = l > 0.f ? 1.f / l : 0.f;
+  if (a.gate != nullptr) f *= sigmoid_f(to_f(static_cast<const bf16*>(a.gate)[row * a.gate_stride + head]));
+  bf16* out = static_cast<bf16*>(a.out) + (row * a.heads + head) * a.kv_rank;
+  for (int i = threadIdx.x * 4; i < a.kv_rank; i += 128 * 4) {
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    for (int c = c0; c <= c1; ++c) {
+      const long long s = ((long long)c * 2 + (c * per >= b0 ? 0 : 1)) * a.heads + head;
+      const float w = exp2f(a.part_ml[s * 2] - m);
+      float v[4];
+      load_n<4>(a.part_o + s * a.kv_rank + i, v);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) acc[j] += w * v[j];
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j) acc[j] *= f;
+    store_n<4>(out + i, acc);
+  }
+}
+
+template <int KS, int MB>
+cudaError_t launch_t(const LatentAttentionArgs& a, cudaStream_t s) {
+  constexpr int M = 16 * MB;
+  constexpr int smem = 2 * KT * KS * 8 * 16 + 4 * M * kSPad * 4 + M * KT * 2 + 2 * M * 4 + 16 * 4;
+  static_assert(smem <= 227 * 1024, "shared memory plan exceeds the SM");
+  cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<KS, MB>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  if (e != cudaSuccess) return e;
+  latent_decode_kernel<KS, MB><<<dim3((unsigned)a.n_cta, (unsigned)((a.heads + M - 1) / M)), kThreads, smem, s>>>(a);
+  latent_decode_merge_kernel<<<dim3((unsigned)a.rows, (unsigned)a.heads), 128, 0, s>>>(a);
+  return cudaGetLastError();
+}
+
+int ks_of(int D) { return D <= 128 ? 2 : (D <= 192 ? 3 : (D <= 320 ? 5 : 9)); }
+
+}  // namespace
+
+bool latent_decode_supported(const LatentAttentionArgs& a) {
+  return a.kv_rank % 8 == 0 && a.rot_dim % 8 == 0 && a.rot_dim > 0 && a.kv_rank + a.rot_dim <= 576 && a.pool_stride % 8 == 0 &&
+         a.rows < (1ll << 30) && (reinterpret_cast<uintptr_t>(a.pool) & 15) == 0 && (reinterpret_cast<uintptr_t>(a.q_abs) & 15) == 0 &&
+         (reinterpret_cast<uintptr_t>(a.out) & 15) == 0;
+}
+
+int latent_decode_ctas(int heads, int sm_count) {
+  const int blocks = heads <= 16 ? 1 : (heads + 31) / 32;
+  const int n = sm_count / blocks;
+  return n > 0 ? n : 1;
+}
+
+cudaError_t launch_latent_decode(const LatentAttentionArgs& a, cudaStream_t s) {
+  if (a.rows == 0) return cudaSuccess;
+  const int ks = ks_of(a.kv_rank + a.rot_dim);
+  if (a.heads <= 16) {
+    if (ks == 2) return launch_t<2, 1>(a, s);
+    if (ks == 3) return launch_t<3, 1>(a, s);
+    if (ks == 5) return launch_t<5, 1>(a, s);
+    return launch_t<9, 1>(a, s);
+  }
+  if (ks == 2) return launch_t<2, 2>(a, s);
+  if (ks == 3) return launch_t<3, 2>(a, s);
+  if (ks == 5) return launch_t<5, 2>(a, s);
+  return launch_t<9, 2>(a, s);
+}
+
+}  // namespace hybrid
+}  // namespace fa

@@ -21,10 +21,9 @@ struct LightningArgs {
   long long total;           // tokens
   void* out;                 // T [tokens, heads * dv]
   int* status;
-  float* seg_state;          // scratch of the segmented prompt kernel: [segments, heads, dk, dv]
-  const int32_t* seg_seq;    // [n_seg] sequence of every segment
-  const int32_t* seg_tok;    // [n_seg] first token of every segment
-  int n_seg, seg_len, max_seg_per_seq;
+  // chunked prompt kernel: a sequence is cut into segments of seg_len tokens that run side by side
+  float* seg_state;          // scratch [n_seq, max_segs, heads, dk, dv] (max_segs > 1 only)
+  int seg_len, max_segs;
 };
 
 // Token-by-token kernel: any size, both types; prompts and decode steps.
@@ -32,6 +31,13 @@ template <typename T> cudaError_t launch_lightning_scan(const LightningArgs& a, 
 // One token per sequence; dv a multiple of 4 and at most 1024.
 template <typename T> cudaError_t launch_lightning_decode(const LightningArgs& a, int sm_count, cudaStream_t s);
 bool lightning_decode_supported(const LightningArgs& a);
+
+
+// Prompts in chunks on the tensor cores (bfloat16; dk <= 128, dk and dv multiples of 8).
+// Segments per sequence and their length (a multiple of the chunk) for the longest sequence of a call.
+int lightning_segments(int n_seq, int heads, int dv, int max_len, int sm_count, int* seg_len);
+bool lightning_chunk_supported(const LightningArgs& a);
+cudaError_t launch_lightning_chunk(const LightningArgs& a, cudaStream_t s);
 
 }  // namespace hybrid
 }  // namespace fa

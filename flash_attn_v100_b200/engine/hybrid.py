@@ -62,7 +62,7 @@ class LightningMixer:
         s, w = self.spec, self.w
         z = linear(h, w["w_in"])                                     # q | k | v | output gate
         o = hops.lightning(z, w["in_at"][:3], s.heads, s.dim, s.vdim, w["decay"], store, step.state_rows, step.starts, step.status,
-                           cu_seqlens=step.cu)
+                           cu_seqlens=step.cu, max_len=max(step.lens) if step.cu is not None else 1)
         at = w["in_at"][3]
         return linear(hops.gated_norm(o, z[:, at:at + s.heads * s.vdim], w["norm"], self.eps), w["w_out"])
 

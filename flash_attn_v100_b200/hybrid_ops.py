@@ -28,6 +28,10 @@ def _check(t, name, dtype, contiguous=True):
         raise RuntimeError(f"{name} must be contiguous")
 
 
+def _workspace(nbytes, device):
+    return torch.empty(nbytes, dtype=torch.uint8, device=device) if nbytes else None
+
+
 def _type(t, name):
     if t.dtype not in _DTYPE:
         raise RuntimeError(f"{name} must be bfloat16 or float32, got {t.dtype}")
@@ -102,8 +106,9 @@ def side_gate(z, side, tokens, off):
     return out
 
 
-def lightning(qkv, offsets, heads, dk, dv, decay, state, slots, starts, status, *, cu_seqlens=None):
-    """Decayed linear attention over packed prompts (cu_seqlens [n_seq + 1]) or one token per sequence.
+def lightning(qkv, offsets, heads, dk, dv, decay, state, slots, starts, status, *, cu_seqlens=None, max_len=0):
+    """Decayed linear attention over packed prompts (cu_seqlens [n_seq + 1], the longest of max_len tokens) or one token per
+    sequence.
     qkv [tokens, stride], offsets = columns of q, k, v; state [n_slots, heads, dk, dv] fp32, updated in place;
     slots / starts [n_seq].  Returns [tokens, heads * dv]."""
     T = _type(qkv, "qkv")
@@ -123,9 +128,12 @@ def lightning(qkv, offsets, heads, dk, dv, decay, state, slots, starts, status, 
         raise RuntimeError("starts must have one entry per sequence")
     tokens = qkv.size(0)
     out = torch.empty((tokens, heads * dv), dtype=T, device=qkv.device)
-    _lib.check_hybrid(_lib.load_hybrid().fah_lightning(
-        _p(qkv), qkv.size(1), *offsets, heads, dk, dv, _p(decay), _p(state), state.size(0), _p(slots), _p(starts), _p(cu_seqlens), n_seq,
-        tokens, _p(out), _p(status), _DTYPE[T], _stream(qkv)))
+    lib, ws = _lib.load_hybrid(), None
+    if cu_seqlens is not None:
+        ws = _workspace(lib.fah_lightning_workspace(n_seq, heads, dk, dv, max_len, _DTYPE[T]), qkv.device)
+    _lib.check_hybrid(lib.fah_lightning(
+        _p(qkv), qkv.size(1), *offsets, heads, dk, dv, _p(decay), _p(state), state.size(0), _p(slots), _p(starts), _p(cu_seqlens), n_seq, max_len,
+        tokens, _p(out), _p(ws), ws.numel() if ws is not None else 0, _p(status), _DTYPE[T], _stream(qkv)))
     return out
 
 
@@ -192,10 +200,12 @@ def latent_attention(q_abs, q, q_off, cos, sin, pool, block_table, tok_seq, posi
         if gate.shape != (rows, heads) or gate.stride(1) != 1:
             raise RuntimeError("gate must be [rows, heads] with contiguous rows")
     out = torch.empty_like(q_abs)
-    _lib.check_hybrid(_lib.load_hybrid().fah_latent_attention(
+    lib = _lib.load_hybrid()
+    ws = _workspace(lib.fah_latent_attention_workspace(heads, kv_rank, rot_dim, rows, _DTYPE[T]), q_abs.device)
+    _lib.check_hybrid(lib.fah_latent_attention(
         _p(q_abs), _p(q), q.size(2), q_off, _p(cos), _p(sin), _p(pool), pool.size(2), pool.size(0), _p(block_table), block_table.size(1),
         block_table.size(0), _p(tok_seq), _p(positions), _p(gate), gate.stride(0) if gate is not None else 0, heads, kv_rank, rot_dim, scale,
-        _p(out), rows, _p(status), _DTYPE[T], _stream(q_abs)))
+        _p(out), rows, _p(ws), ws.numel() if ws is not None else 0, _p(status), _DTYPE[T], _stream(q_abs)))
     return out
 
 

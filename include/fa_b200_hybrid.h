@@ -41,10 +41,13 @@ int fah_side_gate(const void* z, const void* side, const int64_t* tokens, int vo
 
 /* Decayed linear attention with SiLU on q, k, v: per head S = decay * S + k v^T, o = S^T q.
  * qkv [tokens, stride] with the heads x dk queries at column off_q, keys at off_k, heads x dv values at off_v;
- * state [n_slots, heads, dk, dv] fp32; out [tokens, heads * dv].  cu_seqlens null: one token per sequence. */
+ * state [n_slots, heads, dk, dv] fp32; out [tokens, heads * dv].  cu_seqlens null: one token per sequence.
+ * Prompts (cu_seqlens given) take a workspace of fah_lightning_workspace bytes; max_len is the longest sequence of the call. */
+size_t fah_lightning_workspace(int n_seq, int heads, int dk, int dv, int max_len, int dtype);
 int fah_lightning(const void* qkv, int64_t stride, int off_q, int off_k, int off_v, int heads, int dk, int dv, const float* decay,
                   float* state, int n_slots, const int32_t* slots, const int32_t* starts, const int32_t* cu_seqlens, int n_seq,
-                  int64_t tokens, void* out, int32_t* status, int dtype, void* stream);
+                  int max_len, int64_t tokens, void* out, void* workspace, size_t workspace_bytes, int32_t* status, int dtype,
+                  void* stream);
 
 /* down [rows, down_stride]: the query latent at off_q, the key/value latent at off_kv and the shared key part at off_r.
  * cq [rows, q_rank] and the latent c are RMS-normed, the shared part is rotated with cos / sin [rows, rot_dim / 2]; (c, rotated
@@ -62,11 +65,14 @@ int fah_rotate_heads(void* q, const float* cos_t, const float* sin_t, int64_t ro
 
 /* Attention over cached latent rows: every row of (q_abs [rows, heads, kv_rank] | rotated columns
  * [q_off, q_off + rot_dim) of q [rows, heads, q_stride]) sees the keys 0 .. positions[row] of its sequence; values are the
- * latents; the result times sigmoid(gate[row, head]) (gate may be null) goes to out [rows, heads, kv_rank]. */
+ * latents; the result times sigmoid(gate[row, head]) (gate may be null) goes to out [rows, heads, kv_rank].  The workspace has
+ * fah_latent_attention_workspace bytes (0: none is needed). */
+size_t fah_latent_attention_workspace(int heads, int kv_rank, int rot_dim, int64_t rows, int dtype);
 int fah_latent_attention(const void* q_abs, const void* q, int q_stride, int q_off, const float* cos_t, const float* sin_t,
                          const void* pool, int pool_stride, int n_blocks, const int32_t* block_table, int max_blocks, int n_seq,
                          const int32_t* tok_seq, const int32_t* positions, const void* gate, int64_t gate_stride, int heads,
-                         int kv_rank, int rot_dim, float scale, void* out, int64_t rows, int32_t* status, int dtype, void* stream);
+                         int kv_rank, int rot_dim, float scale, void* out, int64_t rows, void* workspace, size_t workspace_bytes,
+                         int32_t* status, int dtype, void* stream);
 
 /* Prompt attention on expanded latents (bfloat16): q [total_q, heads, dim + rot_dim] rotated, kv [total_kv, heads * dim | heads *
  * vdim], kr [total_kv, rot_dim] shared by the heads.  A sequence's queries are its last keys; causal.  The result times
