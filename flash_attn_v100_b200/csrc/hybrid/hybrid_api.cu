@@ -103,7 +103,7 @@ int fah_side_gate(const void* z, const void* side, const int64_t* tokens, int vo
 size_t fah_lightning_workspace(int n_seq, int heads, int dk, int dv, int max_len, int dtype) {
   if (dtype != FAH_BF16 || n_seq <= 0 || heads <= 0 || dk <= 0 || dv <= 0 || max_len <= 0) return 0;
   int seg_len = 0;
-  const int segs = fa::hybrid::lightning_segments(n_seq, heads, dv, max_len, sm_count(), &seg_len);
+  const int segs = fa::hybrid::lightning_segments(n_seq, heads, dk, dv, max_len, sm_count(), &seg_len);
   return segs > 1 ? (size_t)n_seq * segs * heads * dk * dv * sizeof(float) : 0;
 }
 
@@ -130,7 +130,7 @@ int fah_lightning(const void* qkv, int64_t stride, int off_q, int off_k, int off
     const size_t need = fah_lightning_workspace(n_seq, heads, dk, dv, max_len, dtype);
     FAH_REQUIRE(workspace_bytes >= need && (need == 0 || (workspace != nullptr && (reinterpret_cast<uintptr_t>(workspace) & 15) == 0)),
                 "the workspace has %zu bytes, %zu (16-byte aligned) are needed", workspace_bytes, need);
-    a.max_segs = fa::hybrid::lightning_segments(n_seq, heads, dv, max_len, sm_count(), &a.seg_len);
+    a.max_segs = fa::hybrid::lightning_segments(n_seq, heads, dk, dv, max_len, sm_count(), &a.seg_len);
     a.seg_state = static_cast<float*>(workspace);
     return done(fa::hybrid::launch_lightning_chunk(a, st(stream)), "lightning_chunk");
   }
@@ -191,7 +191,9 @@ int fah_latent_attention(const void* q_abs, const void* q, int q_stride, int q_o
     a.part_o = static_cast<float*>(workspace);
     a.part_ml = a.part_o + (int64_t)a.n_cta * 2 * heads * kv_rank;
     a.row_tiles = reinterpret_cast<int32_t*>(a.part_ml + (int64_t)a.n_cta * 2 * heads * 2);
-    return done(fa::hybrid::launch_latent_decode(a, st(stream)), "latent_decode");
+    void* enc = tensor_map_encode();
+    if (enc == nullptr) return fail(FAH_ERR_CUDA, "cuTensorMapEncodeTiled is not available from the driver");
+    return done(fa::hybrid::launch_latent_decode(a, enc, st(stream)), "latent_decode");
   }
   return done(FAH_DISPATCH(dtype, fa::hybrid::launch_latent_attention, a, st(stream)), "latent_attention");
 }

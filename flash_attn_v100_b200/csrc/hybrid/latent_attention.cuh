@@ -38,7 +38,7 @@ template <typename T> cudaError_t launch_latent_attention(const LatentAttentionA
 // Tensor cores (bfloat16; kv_rank + rot_dim <= 576, both multiples of 8).
 bool latent_decode_supported(const LatentAttentionArgs& a);
 int latent_decode_ctas(int heads, int sm_count);   // per head block
-cudaError_t launch_latent_decode(const LatentAttentionArgs& a, cudaStream_t s);
+cudaError_t launch_latent_decode(const LatentAttentionArgs& a, void* encode_fn, cudaStream_t s);   // cuTensorMapEncodeTiled
 
 }  // namespace hybrid
 }  // namespace fa

@@ -7,7 +7,8 @@
 //
 // Eight warps.  Scores: warp = (half of the tile's keys) x (quarter of the columns); its quarter of Q stays in registers for
 // the whole row, and the four partial score tiles are added up in shared memory by the softmax.  Values: warp = an eighth of the
-// latent's columns.  The next tile is copied (cp.async) while the current one is computed.
+// latent's columns.  Warp 0 fetches the next tile by TMA (one box of 16 rows x 64 columns per page and slab, 128-byte swizzle)
+// while the current one is computed.  The wait for a tile is bounded; one that runs out sets the status word.
 #include <math_constants.h>
 
 #include "../common.cuh"
@@ -18,13 +19,22 @@ namespace fa {
 namespace hybrid {
 namespace {
 
+typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
+                                  const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion,
+                                  CUtensorMapFloatOOBfill);
+
 constexpr int KT = 64;         // keys per tile
 constexpr int kThreads = 256;
-constexpr int kSPad = KT + 4;  // row stride of the partial score tiles
+constexpr int kSPad = KT + 8;  // row stride of the partial score tiles
+constexpr int kSlab = KT * 128;
 
-// Unit (16 bytes) `u` of key row `row`, swizzled within groups of eight units.
+// Unit (16 bytes) `u` of key `key`: 128-byte-swizzled slabs of 64 columns.
+__device__ __forceinline__ uint32_t key_off(int key, int u) {
+  return (uint32_t)((u >> 3) * kSlab + key * 128 + ((u ^ key) & 7) * 16);
+}
+// Unit `u` of query row `row`, rows of UNITS units.
 template <int UNITS>
-__device__ __forceinline__ uint32_t key_off(int row, int u) {
+__device__ __forceinline__ uint32_t q_off(int row, int u) {
   return (uint32_t)((row * UNITS + ((u & ~7) | ((u ^ row) & 7))) * 16);
 }
 
@@ -49,22 +59,33 @@ __device__ __forceinline__ int block_scan(int v, int* buf) {
   return v + add;
 }
 
-// KS: 16-column steps per warp quarter (4 * 16 * KS >= kv_rank + rot_dim); MB: 16-head blocks.
+// Partial score tiles; the staged query rows of a new row use the same place.
+__host__ __device__ constexpr int score_bytes(int ks, int mb) {
+  const int s = 4 * 16 * mb * kSPad * 4, q = 16 * mb * ks * 8 * 16;
+  return s > q ? s : q;
+}
+
+// KS: slabs of 64 columns = 16-column steps per warp quarter (4 * 16 * KS >= kv_rank + rot_dim); MB: 16-head blocks.
 template <int KS, int MB>
-__global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const LatentAttentionArgs a) {
+__global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid_constant__ CUtensorMap pool_map,
+                                                                    const LatentAttentionArgs a) {
   constexpr int UNITS = KS * 8;                    // 16-byte units per key row
-  constexpr int STAGE = KT * UNITS * 16;
+  constexpr int STAGE = KS * kSlab;
   constexpr int M = 16 * MB;
+  constexpr int SBYTES = score_bytes(KS, MB);
   constexpr int TPR = kThreads / M;                // softmax threads per row
   constexpr int KPT = KT / TPR;                    // keys per softmax thread
-  extern __shared__ __align__(1024) uint8_t sm[];
+  extern __shared__ uint8_t sm_dyn[];
+  uint8_t* sm = sm_dyn + ((1024u - (smem_u32(sm_dyn) & 1023u)) & 1023u);
   const uint32_t sKV = smem_u32(sm);
   float* sS = reinterpret_cast<float*>(sm + 2 * STAGE);            // [4][M][kSPad]
-  const uint32_t sP = smem_u32(sS + 4 * M * kSPad);                // [M][KT] bfloat16, swizzled
-  float* sAlpha = reinterpret_cast<float*>(sm + 2 * STAGE + 4 * M * kSPad * 4 + M * KT * 2);   // [M]
+  const uint32_t sQ = smem_u32(sS);                                // [M][UNITS] units, while a row starts
+  const uint32_t sP = sQ + SBYTES;                                 // [M][KT] bfloat16, swizzled
+  float* sAlpha = reinterpret_cast<float*>(sm + 2 * STAGE + SBYTES + M * KT * 2);   // [M]
   float* sL = sAlpha + M;                                          // [M]
   int* scan_buf = reinterpret_cast<int*>(sL + M);                  // [8]
   int* found = scan_buf + 8;                                       // [2] first row, its first unit
+  const uint32_t bars = smem_u32(scan_buf + 12);                   // [2] tile has landed
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
   const int cta = blockIdx.x, h0 = blockIdx.y * M;
   const int R = a.kv_rank, D = R + a.rot_dim;
@@ -98,35 +119,43 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const Latent
     }
   }
   const int first_row = found[0];
-  struct Cursor { int row, tile, tiles; };
-  auto start_row = [&](Cursor& c, int row) { c.row = row; c.tile = 0; c.tiles = row_tiles_of(a, row); };
+  if (tid == 0) {
+    mbar_init(bars, 1);
+    mbar_init(bars + 8, 1);
+    mbar_fence_init();
+    fence_proxy_async();
+    tma_prefetch_desc(&pool_map);
+  }
+  __syncthreads();
+  struct Cursor { int row, tile, tiles, n; };
+  auto start_row = [&](Cursor& c, int row) { c.row = row; c.tile = 0; c.n = a.positions[row] + 1; c.tiles = c.n > 0 ? (c.n + KT - 1) / KT : 1; };
   auto advance = [&](Cursor& c) {
     if (++c.tile == c.tiles && c.row + 1 < a.rows) start_row(c, c.row + 1);
   };
 
-  // ---- copies -----------------------------------------------------------------------------------
-  bool bad = false;
-  // lane 0-3 of every warp: pages of the cursor's tile
+  // ---- copies (warp 0) ----------------------------------------------------------------------------
+  bool bad = false, late = false;
+  // lanes 0-3: pages of the cursor's tile (-1: no keys there, -2: not a page of a request); checked when they are used
   auto tile_pages = [&](const Cursor& c) {
-    int page = -1;
-    const int seq = a.tok_seq[c.row], n = a.positions[c.row] + 1, key = c.tile * KT + lane * 16;
-    if (lane < 4 && key < n) {
-      if (seq >= 0 && seq < a.n_seq && (key >> 4) < a.max_blocks) page = a.block_table[(long long)seq * a.max_blocks + (key >> 4)];
-      if (page < 0 || page >= a.n_blocks) { page = -1; bad = true; }
-    }
-    return page;
+    const int seq = a.tok_seq[c.row], key = c.tile * KT + lane * 16;
+    if (lane >= 4 || (key >= c.n && lane > 0)) return -1;
+    if (seq < 0 || seq >= a.n_seq || c.n <= 0 || (key >> 4) >= a.max_blocks) return -2;
+    return a.block_table[(long long)seq * a.max_blocks + (key >> 4)];
   };
-  auto copy_tile = [&](const Cursor& c, int page, int stage) {
-    const int n = a.positions[c.row] + 1 - c.tile * KT;     // keys of the tile that exist
-    const bf16* pool = static_cast<const bf16*>(a.pool);
+  auto copy_tile = [&](int page, int stage) {
+    const bool wrong = lane < 4 && page != -1 && (page < 0 || page >= a.n_blocks);
+    bad |= wrong;
+    if (wrong) page = 0;
+    const int p0 = __shfl_sync(0xffffffffu, page, 0);
+    if (page < 0) page = p0;                        // keys past the end: any page, their weights are zero
+    if (lane == 0) mbar_expect_tx(bars + 8 * stage, STAGE);
+    __syncwarp();
 #pragma unroll
-    for (int i = 0; i < KT * UNITS / kThreads; ++i) {
-      const int idx = tid + i * kThreads, key = idx / UNITS, u = idx - key * UNITS;
-      // the page's owner lane differs within a warp only where a warp's units straddle two rows
-      const int pg = __shfl_sync(0xffffffffu, page, key >> 4);
-      const bool ok = pg >= 0 && key < n && u * 8 < a.pool_stride;
-      const bf16* src = pool + ((long long)(ok ? pg : 0) * 16 + (key & 15)) * a.pool_stride + (ok ? u * 8 : 0);
-      cp_async_16(sKV + stage * STAGE + key_off<UNITS>(key, u), src, ok);
+    for (int b = 0; b < 4 * KS; b += 32) {
+      const int i = b + lane, slab = i % KS, quarter = i / KS;
+      const int pg = __shfl_sync(0xffffffffu, page, quarter & 3);
+      if (i < 4 * KS)
+        tma_load_2d_nohint(sKV + stage * STAGE + slab * kSlab + quarter * 2048, &pool_map, slab * 64, pg * 16, bars + 8 * stage);
     }
   };
 
@@ -134,35 +163,41 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const Latent
   const int slice = warp & 3, khalf = warp >> 2;
   uint32_t qf[MB][KS][4];
   float o[MB][KS][4];
-  auto q_elem = [&](long long row, int head, int c) -> float {
-    if (head >= a.heads || c >= D) return 0.f;
-    if (c < R) return to_f(static_cast<const bf16*>(a.q_abs)[(row * a.heads + head) * R + c]);
-    const int half = a.rot_dim / 2, i = c - R, f = i < half ? i : i - half;
-    const bf16* qr = static_cast<const bf16*>(a.q) + (row * a.heads + head) * a.q_stride + a.q_off;
-    const float cs = a.cos_t[row * half + f], sn = a.sin_t[row * half + f];
-    return i < half ? to_f(qr[i]) * cs - to_f(qr[i + half]) * sn : to_f(qr[i]) * cs + to_f(qr[i - half]) * sn;
-  };
+  // All threads; the score tiles are not in use.  Ends with the fragments in registers, but without a barrier behind it.
   auto load_q = [&](long long row) {
-#pragma unroll
-    for (int m = 0; m < MB; ++m)
-#pragma unroll
-      for (int k = 0; k < KS; ++k)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int head = h0 + m * 16 + g + (e & 1) * 8, c = (slice * KS + k) * 16 + t4 * 2 + (e >> 1) * 8;
-          if (c + 1 < R && head < a.heads)         // two latent columns at once (kv_rank is a multiple of 8)
-            qf[m][k][e] = *reinterpret_cast<const uint32_t*>(static_cast<const bf16*>(a.q_abs) + (row * a.heads + head) * R + c);
-          else
-            qf[m][k][e] = pack_bf162(q_elem(row, head, c), q_elem(row, head, c + 1));
+    const int half = a.rot_dim / 2;
+#pragma unroll 1
+    for (int idx = tid; idx < M * UNITS; idx += kThreads) {
+      const int m = idx / UNITS, u = idx - m * UNITS, c = u * 8, head = h0 + m;
+      uint4 v = make_uint4(0, 0, 0, 0);
+      if (head < a.heads) {
+        if (c < R) {
+          v = *reinterpret_cast<const uint4*>(static_cast<const bf16*>(a.q_abs) + (row * a.heads + head) * R + c);
+        } else if (c < D) {
+          const bf16* qr = static_cast<const bf16*>(a.q) + (row * a.heads + head) * a.q_stride + a.q_off;
+          float e[8];
+#pragma unroll 1
+          for (int j = 0; j < 8; ++j) {
+            const int i = c - R + j, f = i < half ? i : i - half;
+            const float cs = a.cos_t[row * half + f], sn = a.sin_t[row * half + f];
+            e[j] = i < half ? to_f(qr[i]) * cs - to_f(qr[i + half]) * sn : to_f(qr[i]) * cs + to_f(qr[i - half]) * sn;
+          }
+          v = make_uint4(pack_bf162(e[0], e[1]), pack_bf162(e[2], e[3]), pack_bf162(e[4], e[5]), pack_bf162(e[6], e[7]));
         }
+      }
+      asm volatile("st.shared.v4.b32 [%0], {%1,%2,%3,%4};" ::"r"(sQ + q_off<UNITS>(m, u)), "r"(v.x), "r"(v.y), "r"(v.z), "r"(v.w) : "memory");
+    }
+    __syncthreads();
 #pragma unroll
     for (int m = 0; m < MB; ++m)
 #pragma unroll
-      for (int n = 0; n < KS; ++n)
+      for (int k = 0; k < KS; ++k) {
+        ldmatrix_x4(qf[m][k], sQ + q_off<UNITS>(m * 16 + (lane & 15), (slice * KS + k) * 2 + (lane >> 4)));
 #pragma unroll
-        for (int e = 0; e < 4; ++e) o[m][n][e] = 0.f;
+        for (int e = 0; e < 4; ++e) o[m][k][e] = 0.f;
+      }
   };
-  const int srow = tid / TPR, sk0 = (tid % TPR) * KPT;       // softmax: my head row and first key
+  const int srow = tid / TPR, sk0 = (tid % TPR) * 4;         // softmax: my head row; keys sk0 + 4 TPR i .. + 3
   float m_run = -CUDART_INF_F, l_run = 0.f;
   const float sc = a.scale * 1.4426950408889634f;
 
@@ -171,27 +206,28 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const Latent
   cur.tile = u0 - found[1];
   Cursor nxt = cur;
   int piece_tile0 = cur.tile;
-  copy_tile(nxt, tile_pages(nxt), 0);
-  cp_async_commit();
   int page_next = -1;
-  if (u0 + 1 < u1) {
-    advance(nxt);
-    page_next = tile_pages(nxt);
+  if (warp == 0) {
+    copy_tile(tile_pages(nxt), 0);
+    if (u0 + 1 < u1) {
+      advance(nxt);
+      page_next = tile_pages(nxt);
+    }
   }
   load_q(cur.row);
 
+#pragma unroll 1
   for (int u = u0; u < u1; ++u) {
     const int stage = (u - u0) & 1;
-    cp_async_wait<0>();
-    __syncthreads();                                // tile u has landed; the other stage is no longer read
-    if (u + 1 < u1) {
-      copy_tile(nxt, page_next, stage ^ 1);
-      cp_async_commit();
+    __syncthreads();                                // the other stage and the score tiles are no longer read
+    if (warp == 0 && u + 1 < u1) {
+      copy_tile(page_next, stage ^ 1);
       if (u + 2 < u1) {
         advance(nxt);
         page_next = tile_pages(nxt);
       }
     }
+    if (!late) late = !mbar_wait(bars + 8 * stage, (uint32_t)((u - u0) >> 1) & 1u);
     // ---- partial scores -------------------------------------------------------------------------
     {
       float s[MB][4][4];
@@ -207,7 +243,7 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const Latent
         for (int n2 = 0; n2 < 2; ++n2) {
           uint32_t b[4];
           const int key = khalf * 32 + n2 * 16 + (lane & 7) + (lane >> 4) * 8;
-          ldmatrix_x4(b, sKV + stage * STAGE + key_off<UNITS>(key, (slice * KS + k) * 2 + ((lane >> 3) & 1)));
+          ldmatrix_x4(b, sKV + stage * STAGE + key_off(key, (slice * KS + k) * 2 + ((lane >> 3) & 1)));
 #pragma unroll
           for (int m = 0; m < MB; ++m) {
             mma_bf16_16816(s[m][n2 * 2], qf[m][k], b[0], b[1]);
@@ -227,39 +263,39 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const Latent
     __syncthreads();
     // ---- softmax of my row's keys ---------------------------------------------------------------
     {
-      const int valid = a.positions[cur.row] + 1 - cur.tile * KT;
+      const int valid = cur.n - cur.tile * KT;
       float p[KPT];
       float mx = -CUDART_INF_F;
 #pragma unroll
       for (int i = 0; i < KPT; i += 4) {
-        float4 v = *reinterpret_cast<const float4*>(sS + srow * kSPad + sk0 + i);
+        const int c = sk0 + i * TPR;
+        float4 v = *reinterpret_cast<const float4*>(sS + srow * kSPad + c);
 #pragma unroll
         for (int q = 1; q < 4; ++q) {
-          const float4 w = *reinterpret_cast<const float4*>(sS + (q * M + srow) * kSPad + sk0 + i);
+          const float4 w = *reinterpret_cast<const float4*>(sS + (q * M + srow) * kSPad + c);
           v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w;
         }
-        p[i] = v.x; p[i + 1] = v.y; p[i + 2] = v.z; p[i + 3] = v.w;
-      }
-#pragma unroll
-      for (int i = 0; i < KPT; ++i) {
-        p[i] = sk0 + i < valid ? p[i] * sc : -CUDART_INF_F;
-        mx = fmaxf(mx, p[i]);
+        p[i] = c < valid ? v.x * sc : -CUDART_INF_F;
+        p[i + 1] = c + 1 < valid ? v.y * sc : -CUDART_INF_F;
+        p[i + 2] = c + 2 < valid ? v.z * sc : -CUDART_INF_F;
+        p[i + 3] = c + 3 < valid ? v.w * sc : -CUDART_INF_F;
+        mx = fmaxf(fmaxf(mx, fmaxf(p[i], p[i + 1])), fmaxf(p[i + 2], p[i + 3]));
       }
 #pragma unroll
       for (int w = 1; w < TPR; w <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, w));
       const float m_new = fmaxf(m_run, mx);
       const float ref = m_new == -CUDART_INF_F ? 0.f : m_new;
-      const float alpha = exp2f(m_run - ref);       // 0 at the row's first tile
+      const float alpha = fast_exp2(m_run - ref);   // 0 at the row's first tile
       float sum = 0.f;
 #pragma unroll
-      for (int i = 0; i < KPT; ++i) { p[i] = exp2f(p[i] - ref); sum += p[i]; }
+      for (int i = 0; i < KPT; ++i) { p[i] = fast_exp2(p[i] - ref); sum += p[i]; }
 #pragma unroll
       for (int w = 1; w < TPR; w <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, w);
       l_run = l_run * alpha + sum;
       m_run = m_new;
 #pragma unroll
       for (int i = 0; i < KPT; i += 4) {
-        const int c = sk0 + i;
+        const int c = sk0 + i * TPR;
         const uint32_t addr = sP + (uint32_t)((srow * 8 + ((c >> 3) ^ (srow & 7))) * 16 + (c & 7) * 2);
         asm volatile("st.shared.v2.b32 [%0], {%1,%2};" ::"r"(addr), "r"(pack_bf162(p[i], p[i + 1])), "r"(pack_bf162(p[i + 2], p[i + 3]))
                      : "memory");
@@ -291,7 +327,7 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const Latent
         for (int n = 0; n < KS; ++n) {
           if ((warp * KS + n) * 8 < R) {
             uint32_t b[4];
-            ldmatrix_x4_trans(b, sKV + stage * STAGE + key_off<UNITS>(k2 * 32 + lane, warp * KS + n));
+            ldmatrix_x4_trans(b, sKV + stage * STAGE + key_off(k2 * 32 + lane, warp * KS + n));
 #pragma unroll
             for (int m = 0; m < MB; ++m) {
               mma_bf16_16816(o[m][n], pf[m][0], b[0], b[1]);
@@ -345,7 +381,11 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const Latent
     }
     if (u + 1 < u1) advance(cur);
   }
-  if (bad) atomicOr(a.status, 2);
+  if (bad) atomicOr(a.status, kStatusBadPageId);
+  if (late) {                                       // leave only after another (bounded) wait for the copies in flight
+    atomicOr(a.status, kStatusWaitTimeout);
+    for (int i = u1 - u0 >= 2 ? u1 - 2 : u1 - 1; i < u1; ++i) mbar_wait(bars + 8 * ((i - u0) & 1), (uint32_t)((i - u0) >> 1) & 1u);
+  }
 }
 
 // Rows that several CTAs worked on: log-sum-exp merge of their partial sums.  One CTA per (row, head).
@@ -387,13 +427,13 @@ __global__ void __launch_bounds__(128) latent_decode_merge_kernel(const LatentAt
 }
 
 template <int KS, int MB>
-cudaError_t launch_t(const LatentAttentionArgs& a, cudaStream_t s) {
+cudaError_t launch_t(const LatentAttentionArgs& a, const CUtensorMap& map, cudaStream_t s) {
   constexpr int M = 16 * MB;
-  constexpr int smem = 2 * KT * KS * 8 * 16 + 4 * M * kSPad * 4 + M * KT * 2 + 2 * M * 4 + 16 * 4;
+  constexpr int smem = 1024 + 2 * KS * kSlab + score_bytes(KS, MB) + M * KT * 2 + 2 * M * 4 + 12 * 4 + 2 * 8;
   static_assert(smem <= 227 * 1024, "shared memory plan exceeds the SM");
   cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<KS, MB>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (e != cudaSuccess) return e;
-  latent_decode_kernel<KS, MB><<<dim3((unsigned)a.n_cta, (unsigned)((a.heads + M - 1) / M)), kThreads, smem, s>>>(a);
+  latent_decode_kernel<KS, MB><<<dim3((unsigned)a.n_cta, (unsigned)((a.heads + M - 1) / M)), kThreads, smem, s>>>(map, a);
   latent_decode_merge_kernel<<<dim3((unsigned)a.rows, (unsigned)a.heads), 128, 0, s>>>(a);
   return cudaGetLastError();
 }
@@ -414,19 +454,27 @@ int latent_decode_ctas(int heads, int sm_count) {
   return n > 0 ? n : 1;
 }
 
-cudaError_t launch_latent_decode(const LatentAttentionArgs& a, cudaStream_t s) {
+cudaError_t launch_latent_decode(const LatentAttentionArgs& a, void* encode_fn, cudaStream_t s) {
   if (a.rows == 0) return cudaSuccess;
+  CUtensorMap map;
+  const cuuint64_t dims[2] = {(cuuint64_t)a.pool_stride, (cuuint64_t)a.n_blocks * 16};
+  const cuuint64_t strides[1] = {(cuuint64_t)a.pool_stride * 2};
+  const cuuint32_t box[2] = {64, 16}, estr[2] = {1, 1};
+  if (reinterpret_cast<EncodeTiledFn>(encode_fn)(&map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(a.pool), dims, strides, box, estr,
+                                                 CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                                                 CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
+    return cudaErrorInvalidValue;
   const int ks = ks_of(a.kv_rank + a.rot_dim);
   if (a.heads <= 16) {
-    if (ks == 2) return launch_t<2, 1>(a, s);
-    if (ks == 3) return launch_t<3, 1>(a, s);
-    if (ks == 5) return launch_t<5, 1>(a, s);
-    return launch_t<9, 1>(a, s);
+    if (ks == 2) return launch_t<2, 1>(a, map, s);
+    if (ks == 3) return launch_t<3, 1>(a, map, s);
+    if (ks == 5) return launch_t<5, 1>(a, map, s);
+    return launch_t<9, 1>(a, map, s);
   }
-  if (ks == 2) return launch_t<2, 2>(a, s);
-  if (ks == 3) return launch_t<3, 2>(a, s);
-  if (ks == 5) return launch_t<5, 2>(a, s);
-  return launch_t<9, 2>(a, s);
+  if (ks == 2) return launch_t<2, 2>(a, map, s);
+  if (ks == 3) return launch_t<3, 2>(a, map, s);
+  if (ks == 5) return launch_t<5, 2>(a, map, s);
+  return launch_t<9, 2>(a, map, s);
 }
 
 }  // namespace hybrid

@@ -35,9 +35,12 @@ bool lightning_decode_supported(const LightningArgs& a);
 
 // Prompts in chunks on the tensor cores (bfloat16; dk <= 128, dk and dv multiples of 8).
 // Segments per sequence and their length (a multiple of the chunk) for the longest sequence of a call.
-int lightning_segments(int n_seq, int heads, int dv, int max_len, int sm_count, int* seg_len);
+int lightning_segments(int n_seq, int heads, int dk, int dv, int max_len, int sm_count, int* seg_len);
 bool lightning_chunk_supported(const LightningArgs& a);
-cudaError_t launch_lightning_chunk(const LightningArgs& a, cudaStream_t s);
+cudaError_t launch_lightning_chunk(const LightningArgs& a, cudaStream_t s);   // dk, dv <= 64, mma.sync
+cudaError_t launch_lightning_tc5(const LightningArgs& a, cudaStream_t s);     // larger heads, tcgen05
+// Turns what every segment adds to the state into the state at the start of every segment.
+cudaError_t launch_lightning_segment_scan(const LightningArgs& a, cudaStream_t s);
 
 }  // namespace hybrid
 }  // namespace fa

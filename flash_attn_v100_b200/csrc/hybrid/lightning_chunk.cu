@@ -303,33 +303,27 @@ __global__ void __launch_bounds__(256) lightning_segment_scan_kernel(const Light
   }
 }
 
-template <int DK>
-cudaError_t launch_t(const LightningArgs& a, cudaStream_t stream) {
-  constexpr int smem = (2 * C * DK + C * BV + 2 * DK * BV) * 2 + (C + 1) * 4;
-  const dim3 grid((unsigned)(a.n_seq * a.max_segs), (unsigned)a.heads, (unsigned)((a.dv + BV - 1) / BV));
-  cudaError_t e;
-  if (a.max_segs > 1) {
-    e = cudaFuncSetAttribute(lightning_chunk_kernel<DK, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-    if (e != cudaSuccess) return e;
-    lightning_chunk_kernel<DK, true><<<grid, kThreads, smem, stream>>>(a);
-    lightning_segment_scan_kernel<<<dim3((unsigned)((a.dk * a.dv + 255) / 256), (unsigned)a.heads, (unsigned)a.n_seq), 256, 0, stream>>>(a);
-  }
-  e = cudaFuncSetAttribute(lightning_chunk_kernel<DK, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-  if (e != cudaSuccess) return e;
-  lightning_chunk_kernel<DK, false><<<grid, kThreads, smem, stream>>>(a);
-  return cudaGetLastError();
-}
+constexpr int kBigChunk = 128, kBigCols = 128;     // lightning_tc5.cu
+
+bool big_heads(int dk, int dv) { return dk > 64 || dv > 64; }
 
 }  // namespace
 
-int lightning_segments(int n_seq, int heads, int dv, int max_len, int sm_count, int* seg_len) {
-  // four CTAs per SM (two are resident at a time) where the batch alone does not give two, in segments of at least eight chunks: a segment's
-  // keys and values are read twice, which only pays while SMs would stay empty
-  const long long tasks = (long long)n_seq * heads * ((dv + BV - 1) / BV);
-  long long segs = tasks >= 2ll * sm_count ? 1 : (4ll * sm_count + tasks - 1) / tasks;
+cudaError_t launch_lightning_segment_scan(const LightningArgs& a, cudaStream_t stream) {
+  lightning_segment_scan_kernel<<<dim3((unsigned)((a.dk * a.dv + 255) / 256), (unsigned)a.heads, (unsigned)a.n_seq), 256, 0, stream>>>(a);
+  return cudaGetLastError();
+}
+
+int lightning_segments(int n_seq, int heads, int dk, int dv, int max_len, int sm_count, int* seg_len) {
+  // as many CTAs as run side by side (one per SM of the tcgen05 kernel, two of the other), in segments of at least 512
+  // tokens: a segment's keys and values are read twice, which only pays while SMs would stay empty
+  const bool big = big_heads(dk, dv);
+  const int chunk = big ? kBigChunk : C, slots = (big ? 1 : 2) * sm_count;
+  const long long tasks = (long long)n_seq * heads * ((dv + (big ? kBigCols : BV) - 1) / (big ? kBigCols : BV));
+  const long long segs = tasks * 2 > slots ? 1 : slots / tasks;
   long long len = (max_len + segs - 1) / segs;
-  if (len < 8 * C) len = 8 * C;
-  len = (len + C - 1) / C * C;
+  if (len < 512) len = 512;
+  len = (len + chunk - 1) / chunk * chunk;
   *seg_len = (int)len;
   return (int)((max_len + len - 1) / len);
 }
@@ -339,9 +333,24 @@ bool lightning_chunk_supported(const LightningArgs& a) {
          a.off_v % 8 == 0 && (reinterpret_cast<uintptr_t>(a.qkv) & 15) == 0 && (reinterpret_cast<uintptr_t>(a.out) & 15) == 0;
 }
 
-cudaError_t launch_lightning_chunk(const LightningArgs& a, cudaStream_t s) {
+cudaError_t launch_lightning_chunk(const LightningArgs& a, cudaStream_t stream) {
   if (a.n_seq == 0) return cudaSuccess;
-  return a.dk <= 64 ? launch_t<64>(a, s) : launch_t<128>(a, s);
+  if (big_heads(a.dk, a.dv)) return launch_lightning_tc5(a, stream);
+  constexpr int DK = 64;
+  constexpr int smem = (2 * C * DK + C * BV + 2 * DK * BV) * 2 + (C + 1) * 4;
+  const dim3 grid((unsigned)(a.n_seq * a.max_segs), (unsigned)a.heads, (unsigned)((a.dv + BV - 1) / BV));
+  cudaError_t e;
+  if (a.max_segs > 1) {
+    e = cudaFuncSetAttribute(lightning_chunk_kernel<DK, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return e;
+    lightning_chunk_kernel<DK, true><<<grid, kThreads, smem, stream>>>(a);
+    e = launch_lightning_segment_scan(a, stream);
+    if (e != cudaSuccess) return e;
+  }
+  e = cudaFuncSetAttribute(lightning_chunk_kernel<DK, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  if (e != cudaSuccess) return e;
+  lightning_chunk_kernel<DK, false><<<grid, kThreads, smem, stream>>>(a);
+  return cudaGetLastError();
 }
 
 }  // namespace hybrid

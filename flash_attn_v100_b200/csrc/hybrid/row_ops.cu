@@ -11,10 +11,10 @@ namespace hybrid {
 namespace {
 
 constexpr int kThreads = 256;
-constexpr int kKeep = 8;      // vectors per thread that stay in registers between the passes over a row
 
+// KEEP: vectors per thread that stay in registers between the passes over a row (0: the row is read again).
 // x (+)= [embedding] + [delta or rmsnorm(delta) * delta_w]; out = rmsnorm(x) * w (or x).  One CTA per row.
-template <typename T, int VEC, bool KEEP>
+template <typename T, int VEC, int KEEP>
 __global__ void __launch_bounds__(kThreads) residual_norm_kernel(const ResidualNormArgs a) {
   __shared__ float red[kThreads / 32];
   const long long row = blockIdx.x;
@@ -28,7 +28,7 @@ __global__ void __launch_bounds__(kThreads) residual_norm_kernel(const ResidualN
     e = static_cast<const T*>(a.embed) + tok * a.cols;
   }
   const int nv = a.cols / VEC;
-  float keep[KEEP ? kKeep : 1][VEC];
+  float keep[KEEP > 0 ? KEEP : 1][VEC];
   float dinv = 1.f;
   if (d != nullptr && dw != nullptr) {
     float ss = 0.f;
@@ -68,9 +68,9 @@ __global__ void __launch_bounds__(kThreads) residual_norm_kernel(const ResidualN
   };
   const bool changed = d != nullptr || e != nullptr;
   float ss = 0.f;
-  if constexpr (KEEP) {
+  if constexpr (KEEP > 0) {
 #pragma unroll
-    for (int n = 0; n < kKeep; ++n) {
+    for (int n = 0; n < KEEP; ++n) {
       const int c = threadIdx.x + n * kThreads;
       if (c < nv) {
         updated(c, keep[n]);
@@ -101,9 +101,9 @@ __global__ void __launch_bounds__(kThreads) residual_norm_kernel(const ResidualN
     }
     store_n<VEC>(out + c * VEC, v);
   };
-  if constexpr (KEEP) {
+  if constexpr (KEEP > 0) {
 #pragma unroll
-    for (int n = 0; n < kKeep; ++n) {
+    for (int n = 0; n < KEEP; ++n) {
       const int c = threadIdx.x + n * kThreads;
       if (c < nv) emit(c, keep[n]);
     }
@@ -116,18 +116,18 @@ __global__ void __launch_bounds__(kThreads) residual_norm_kernel(const ResidualN
 }
 
 // out = rmsnorm(o) * w * sigmoid(g), the norm taken over the whole row.  One CTA per row.
-template <typename T, int VEC, bool KEEP>
+template <typename T, int VEC, int KEEP>
 __global__ void __launch_bounds__(kThreads) gated_norm_kernel(const T* o, const T* g, long long g_stride, const T* w, T* out,
                                                              int cols, float eps) {
   __shared__ float red[kThreads / 32];
   const long long row = blockIdx.x;
   o += row * cols; g += row * g_stride; out += row * cols;
   const int nv = cols / VEC;
-  float keep[KEEP ? kKeep : 1][VEC];
+  float keep[KEEP > 0 ? KEEP : 1][VEC];
   float ss = 0.f;
-  if constexpr (KEEP) {
+  if constexpr (KEEP > 0) {
 #pragma unroll
-    for (int n = 0; n < kKeep; ++n) {
+    for (int n = 0; n < KEEP; ++n) {
       const int c = threadIdx.x + n * kThreads;
       if (c < nv) {
         load_n<VEC>(o + c * VEC, keep[n]);
@@ -151,9 +151,9 @@ __global__ void __launch_bounds__(kThreads) gated_norm_kernel(const T* o, const 
     for (int i = 0; i < VEC; ++i) v[i] = v[i] * inv * wv[i] * sigmoid_f(gv[i]);
     store_n<VEC>(out + c * VEC, v);
   };
-  if constexpr (KEEP) {
+  if constexpr (KEEP > 0) {
 #pragma unroll
-    for (int n = 0; n < kKeep; ++n) {
+    for (int n = 0; n < KEEP; ++n) {
       const int c = threadIdx.x + n * kThreads;
       if (c < nv) emit(c, keep[n]);
     }
@@ -287,9 +287,11 @@ cudaError_t launch_residual_norm(const ResidualNormArgs& a, cudaStream_t s) {
   const unsigned g = (unsigned)a.rows;
   const bool vec = a.cols % 4 == 0 && aligned16(a.x) && aligned16(a.delta) && aligned16(a.delta_w) && aligned16(a.embed) &&
                    aligned16(a.w) && aligned16(a.out);
-  if (vec && a.cols <= 4 * kKeep * kThreads) residual_norm_kernel<T, 4, true><<<g, kThreads, 0, s>>>(a);
-  else if (vec) residual_norm_kernel<T, 4, false><<<g, kThreads, 0, s>>>(a);
-  else residual_norm_kernel<T, 1, false><<<g, kThreads, 0, s>>>(a);
+  if (vec && a.cols <= 4 * kThreads) residual_norm_kernel<T, 4, 1><<<g, kThreads, 0, s>>>(a);
+  else if (vec && a.cols <= 16 * kThreads) residual_norm_kernel<T, 4, 4><<<g, kThreads, 0, s>>>(a);
+  else if (vec && a.cols <= 32 * kThreads) residual_norm_kernel<T, 4, 8><<<g, kThreads, 0, s>>>(a);
+  else if (vec) residual_norm_kernel<T, 4, 0><<<g, kThreads, 0, s>>>(a);
+  else residual_norm_kernel<T, 1, 0><<<g, kThreads, 0, s>>>(a);
   return cudaGetLastError();
 }
 
@@ -300,10 +302,12 @@ cudaError_t launch_gated_norm(const void* o, const void* g, long long g_stride, 
   const T *op = static_cast<const T*>(o), *gp = static_cast<const T*>(g), *wp = static_cast<const T*>(w);
   T* outp = static_cast<T*>(out);
   const bool vec = cols % 8 == 0 && g_stride % 8 == 0 && aligned16(o) && aligned16(g) && aligned16(w) && aligned16(out);
-  if (vec && cols <= 8 * kKeep * kThreads)
-    gated_norm_kernel<T, 8, true><<<(unsigned)rows, kThreads, 0, s>>>(op, gp, g_stride, wp, outp, cols, eps);
-  else
-    gated_norm_kernel<T, 1, false><<<(unsigned)rows, kThreads, 0, s>>>(op, gp, g_stride, wp, outp, cols, eps);
+  const unsigned grid = (unsigned)rows;
+  if (vec && cols <= 8 * kThreads) gated_norm_kernel<T, 8, 1><<<grid, kThreads, 0, s>>>(op, gp, g_stride, wp, outp, cols, eps);
+  else if (vec && cols <= 16 * kThreads) gated_norm_kernel<T, 8, 2><<<grid, kThreads, 0, s>>>(op, gp, g_stride, wp, outp, cols, eps);
+  else if (vec && cols <= 32 * kThreads) gated_norm_kernel<T, 8, 4><<<grid, kThreads, 0, s>>>(op, gp, g_stride, wp, outp, cols, eps);
+  else if (vec) gated_norm_kernel<T, 8, 0><<<grid, kThreads, 0, s>>>(op, gp, g_stride, wp, outp, cols, eps);
+  else gated_norm_kernel<T, 1, 0><<<grid, kThreads, 0, s>>>(op, gp, g_stride, wp, outp, cols, eps);
   return cudaGetLastError();
 }
 

@@ -17,11 +17,14 @@ def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--case", default="paged_decode",
                     choices=["paged_decode", "int8_decode", "varlen_prefill", "contig_decode", "int8_kv_decode",
-                             "sliding_window_decode"])
+                             "sliding_window_decode", "latent_decode", "latent_prefill", "lightning_prefill",
+                             "lightning_decode"])
     ap.add_argument("--batch", type=int, default=16)
     ap.add_argument("--iters", type=int, default=3)
     ap.add_argument("--seed", type=int, default=0)
     args = ap.parse_args()
+    if args.case.startswith(("latent", "lightning")):
+        return hybrid(args)
     import flash_attn_v100 as fa
     import flash_attn_v100_b200
     from flash_attn_v100_b200.synthetic import make_paged_tables
@@ -86,6 +89,46 @@ def main():
         run()
     torch.cuda.synchronize()
     flash_attn_v100_b200.check_async_errors()
+    print("done")
+
+
+def hybrid(args):
+    """Kernels of the hybrid decoder: 32 heads of 128 (64 rotated), latent of 512, prompts of 1024 and 4096 cached tokens."""
+    from flash_attn_v100_b200 import hybrid_ops as hops
+    dev = torch.device("cuda", 0)
+    g = torch.Generator(device=dev).manual_seed(args.seed)
+    rnd = lambda *s: torch.randn(*s, generator=g, device=dev).bfloat16()
+    st = torch.zeros(1, dtype=torch.int32, device=dev)
+    H, D, R, L, B = 32, 128, 64, 512, args.batch
+    rows = torch.arange(B, dtype=torch.int32, device=dev)
+    if args.case == "latent_decode":
+        ctx = 4096
+        table = torch.randperm(B * ctx // 16).to(torch.int32).view(B, ctx // 16).to(dev)
+        pool, qa, q, gate = rnd(B * ctx // 16, 16, L + R), rnd(B, H, L), rnd(B, H, D + R), rnd(B, H)
+        cos, sin = (torch.rand(B, R // 2, generator=g, device=dev) for _ in range(2))
+        pos = torch.full((B,), ctx - 1, dtype=torch.int32, device=dev)
+        run = lambda: hops.latent_attention(qa, q, D, cos, sin, pool, table, rows, pos, gate, L, R, 0.07, st)
+        print(f"case latent_decode: B={B} tokens={B * ctx} cache_bytes={B * ctx * (L + R) * 2}")
+    elif args.case == "latent_prefill":
+        n = 1024
+        cu = torch.arange(B + 1, dtype=torch.int32, device=dev) * n
+        q, kv, kr, gate = rnd(B * n, H * (D + R)), rnd(B * n, 2 * H * D), rnd(B * n, R), rnd(B * n, H)
+        run = lambda: hops.latent_prefill(q, kv, kr, gate, cu, cu, n, H, D, D, 0.07, st)
+        print(f"case latent_prefill: seqs={B} flops={B * 2 * H * (2 * D + R) * n * (n + 1) // 2}")
+    else:
+        prompt = args.case == "lightning_prefill"
+        n = 1024 if prompt else 1
+        cu = torch.arange(B + 1, dtype=torch.int32, device=dev) * n if prompt else None
+        z, state = rnd(B * n, 3 * H * D), torch.zeros(B, H, D, D, device=dev)
+        decay = 1.0 - torch.rand(H, generator=g, device=dev) * 0.2
+        starts = torch.full((B,), 0 if prompt else 9, dtype=torch.int32, device=dev)
+        run = lambda: hops.lightning(z, (0, H * D, 2 * H * D), H, D, D, decay, state, rows, starts, st, cu_seqlens=cu, max_len=n)
+        print(f"case {args.case}: seqs={B} row_bytes={B * n * H * D * 8} state_bytes={B * H * D * D * 8}")
+    for _ in range(args.iters + 1):
+        run()
+    torch.cuda.synchronize()
+    if int(st.item()):
+        raise RuntimeError(f"a kernel recorded status {int(st.item())}")
     print("done")
 
 
