@@ -5,9 +5,9 @@
 // 32, the M rows of the MMAs) as key and as value.  The (row, key tile) units of the batch are numbered row by row and cut
 // into equal runs, one per CTA, whatever the lengths; a row that is cut leaves partial sums that a second kernel merges.
 //
-// Eight warps.  Scores: warp = (half of the tile's keys) x (quarter of the columns); its quarter of Q stays in registers for
-// the whole row, and the four partial score tiles are added up in shared memory by the softmax.  Values: warp = an eighth of the
-// latent's columns.  Warp 0 fetches the next tile by TMA (one box of 16 rows x 64 columns per page and slab, 128-byte swizzle)
+// Sixteen warps.  Scores: warp = (a quarter of the tile's keys) x (one 16-column step of every slab); the four partial score
+// tiles are added up in shared memory by the softmax.  Values: warp = 8 columns of
+// every other slab.  (With these shares every shared-memory address is a per-warp base plus a constant.)  Warp 0 fetches the next tile by TMA (one box of 16 rows x 64 columns per page and slab, 128-byte swizzle)
 // while the current one is computed.  The wait for a tile is bounded; one that runs out sets the status word.
 #include <math_constants.h>
 
@@ -24,7 +24,8 @@ typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t,
                                   CUtensorMapFloatOOBfill);
 
 constexpr int KT = 64;         // keys per tile
-constexpr int kThreads = 256;
+constexpr int kThreads = 512;
+constexpr int kWarps = kThreads / 32;
 constexpr int kSPad = KT + 8;  // row stride of the partial score tiles
 constexpr int kSlab = KT * 128;
 
@@ -43,7 +44,7 @@ __device__ __forceinline__ int row_tiles_of(const LatentAttentionArgs& a, long l
   return n > 0 ? (n + KT - 1) / KT : 1;
 }
 
-// Inclusive scan over the block of one int per thread; `buf` holds 8 ints.
+// Inclusive scan over the block of one int per thread; `buf` holds one int per warp.
 __device__ __forceinline__ int block_scan(int v, int* buf) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
 #pragma unroll
@@ -59,12 +60,6 @@ __device__ __forceinline__ int block_scan(int v, int* buf) {
   return v + add;
 }
 
-// Partial score tiles; the staged query rows of a new row use the same place.
-__host__ __device__ constexpr int score_bytes(int ks, int mb) {
-  const int s = 4 * 16 * mb * kSPad * 4, q = 16 * mb * ks * 8 * 16;
-  return s > q ? s : q;
-}
-
 // KS: slabs of 64 columns = 16-column steps per warp quarter (4 * 16 * KS >= kv_rank + rot_dim); MB: 16-head blocks.
 template <int KS, int MB>
 __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid_constant__ CUtensorMap pool_map,
@@ -72,20 +67,20 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
   constexpr int UNITS = KS * 8;                    // 16-byte units per key row
   constexpr int STAGE = KS * kSlab;
   constexpr int M = 16 * MB;
-  constexpr int SBYTES = score_bytes(KS, MB);
-  constexpr int TPR = kThreads / M;                // softmax threads per row
-  constexpr int KPT = KT / TPR;                    // keys per softmax thread
+  constexpr int SBYTES = 4 * M * kSPad * 4, QBYTES = M * UNITS * 16;
+  constexpr int TPR = 16;                          // softmax threads per row, four keys each
+  constexpr int NT = (KS + 1) / 2;                 // 8-column value tiles per warp
   extern __shared__ uint8_t sm_dyn[];
   uint8_t* sm = sm_dyn + ((1024u - (smem_u32(sm_dyn) & 1023u)) & 1023u);
   const uint32_t sKV = smem_u32(sm);
   float* sS = reinterpret_cast<float*>(sm + 2 * STAGE);            // [4][M][kSPad]
-  const uint32_t sQ = smem_u32(sS);                                // [M][UNITS] units, while a row starts
-  const uint32_t sP = sQ + SBYTES;                                 // [M][KT] bfloat16, swizzled
-  float* sAlpha = reinterpret_cast<float*>(sm + 2 * STAGE + SBYTES + M * KT * 2);   // [M]
+  const uint32_t sQ = smem_u32(sS) + SBYTES;                       // [M][UNITS] units: the current row's queries
+  const uint32_t sP = sQ + QBYTES;                                 // [M][KT] bfloat16, swizzled
+  float* sAlpha = reinterpret_cast<float*>(sm + 2 * STAGE + SBYTES + QBYTES + M * KT * 2);   // [M]
   float* sL = sAlpha + M;                                          // [M]
-  int* scan_buf = reinterpret_cast<int*>(sL + M);                  // [8]
-  int* found = scan_buf + 8;                                       // [2] first row, its first unit
-  const uint32_t bars = smem_u32(scan_buf + 12);                   // [2] tile has landed
+  int* scan_buf = reinterpret_cast<int*>(sL + M);                  // [kWarps]
+  int* found = scan_buf + kWarps;                                  // [2] first row, its first unit
+  const uint32_t bars = smem_u32(scan_buf + kWarps + 2);           // [2] tile has landed
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
   const int cta = blockIdx.x, h0 = blockIdx.y * M;
   const int R = a.kv_rank, D = R + a.rot_dim;
@@ -160,10 +155,12 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
   };
 
   // ---- per-row state ----------------------------------------------------------------------------
-  const int slice = warp & 3, khalf = warp >> 2;
-  uint32_t qf[MB][KS][4];
-  float o[MB][KS][4];
-  // All threads; the score tiles are not in use.  Ends with the fragments in registers, but without a barrier behind it.
+  const int slice = warp & 3, kquarter = warp >> 2;
+  // my lane's ldmatrix addresses within a stage (scores: my 16 keys; values: all keys; queries: 16 heads)
+  const uint32_t k_base = key_off(kquarter * 16 + (lane & 7) + (lane >> 4) * 8, slice * 2 + ((lane >> 3) & 1)), v_base = key_off(lane, warp);
+  const uint32_t q_base = sQ + q_off<UNITS>(lane & 15, slice * 2 + (lane >> 4));
+  float o[MB][NT][4];
+  // All threads; a barrier follows before the queries are read.
   auto load_q = [&](long long row) {
     const int half = a.rot_dim / 2;
 #pragma unroll 1
@@ -176,7 +173,7 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
         } else if (c < D) {
           const bf16* qr = static_cast<const bf16*>(a.q) + (row * a.heads + head) * a.q_stride + a.q_off;
           float e[8];
-#pragma unroll 1
+#pragma unroll
           for (int j = 0; j < 8; ++j) {
             const int i = c - R + j, f = i < half ? i : i - half;
             const float cs = a.cos_t[row * half + f], sn = a.sin_t[row * half + f];
@@ -187,17 +184,14 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
       }
       asm volatile("st.shared.v4.b32 [%0], {%1,%2,%3,%4};" ::"r"(sQ + q_off<UNITS>(m, u)), "r"(v.x), "r"(v.y), "r"(v.z), "r"(v.w) : "memory");
     }
-    __syncthreads();
 #pragma unroll
     for (int m = 0; m < MB; ++m)
 #pragma unroll
-      for (int k = 0; k < KS; ++k) {
-        ldmatrix_x4(qf[m][k], sQ + q_off<UNITS>(m * 16 + (lane & 15), (slice * KS + k) * 2 + (lane >> 4)));
+      for (int n = 0; n < NT; ++n)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) o[m][k][e] = 0.f;
-      }
+        for (int e = 0; e < 4; ++e) o[m][n][e] = 0.f;
   };
-  const int srow = tid / TPR, sk0 = (tid % TPR) * 4;         // softmax: my head row; keys sk0 + 4 TPR i .. + 3
+  const int srow = tid / TPR, sk0 = (tid % TPR) * 4;         // softmax: my head row and its four keys
   float m_run = -CUDART_INF_F, l_run = 0.f;
   const float sc = a.scale * 1.4426950408889634f;
 
@@ -230,76 +224,63 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
     if (!late) late = !mbar_wait(bars + 8 * stage, (uint32_t)((u - u0) >> 1) & 1u);
     // ---- partial scores -------------------------------------------------------------------------
     {
-      float s[MB][4][4];
+      float s[MB][2][4];
 #pragma unroll
       for (int m = 0; m < MB; ++m)
 #pragma unroll
-        for (int n = 0; n < 4; ++n)
+        for (int n = 0; n < 2; ++n)
 #pragma unroll
           for (int e = 0; e < 4; ++e) s[m][n][e] = 0.f;
+      const uint32_t kb = sKV + stage * STAGE + k_base;
 #pragma unroll
       for (int k = 0; k < KS; ++k) {
+        uint32_t b[4];
+        ldmatrix_x4(b, kb + k * kSlab);
 #pragma unroll
-        for (int n2 = 0; n2 < 2; ++n2) {
-          uint32_t b[4];
-          const int key = khalf * 32 + n2 * 16 + (lane & 7) + (lane >> 4) * 8;
-          ldmatrix_x4(b, sKV + stage * STAGE + key_off(key, (slice * KS + k) * 2 + ((lane >> 3) & 1)));
-#pragma unroll
-          for (int m = 0; m < MB; ++m) {
-            mma_bf16_16816(s[m][n2 * 2], qf[m][k], b[0], b[1]);
-            mma_bf16_16816(s[m][n2 * 2 + 1], qf[m][k], b[2], b[3]);
-          }
+        for (int m = 0; m < MB; ++m) {
+          uint32_t q[4];
+          ldmatrix_x4(q, q_base + (uint32_t)(m * 16 * UNITS * 16 + k * 128));
+          mma_bf16_16816(s[m][0], q, b[0], b[1]);
+          mma_bf16_16816(s[m][1], q, b[2], b[3]);
         }
       }
 #pragma unroll
       for (int m = 0; m < MB; ++m)
 #pragma unroll
-        for (int n = 0; n < 4; ++n)
+        for (int n = 0; n < 2; ++n)
 #pragma unroll
           for (int h = 0; h < 2; ++h)
-            *reinterpret_cast<float2*>(sS + (slice * M + m * 16 + g + h * 8) * kSPad + khalf * 32 + n * 8 + t4 * 2) =
+            *reinterpret_cast<float2*>(sS + (slice * M + m * 16 + g + h * 8) * kSPad + kquarter * 16 + n * 8 + t4 * 2) =
                 make_float2(s[m][n][2 * h], s[m][n][2 * h + 1]);
     }
     __syncthreads();
     // ---- softmax of my row's keys ---------------------------------------------------------------
-    {
-      const int valid = cur.n - cur.tile * KT;
-      float p[KPT];
-      float mx = -CUDART_INF_F;
+    if (srow < M) {                                 // (whole warps)
+      const int valid = cur.n - cur.tile * KT - sk0;
+      float4 v = *reinterpret_cast<const float4*>(sS + srow * kSPad + sk0);
 #pragma unroll
-      for (int i = 0; i < KPT; i += 4) {
-        const int c = sk0 + i * TPR;
-        float4 v = *reinterpret_cast<const float4*>(sS + srow * kSPad + c);
-#pragma unroll
-        for (int q = 1; q < 4; ++q) {
-          const float4 w = *reinterpret_cast<const float4*>(sS + (q * M + srow) * kSPad + c);
-          v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w;
-        }
-        p[i] = c < valid ? v.x * sc : -CUDART_INF_F;
-        p[i + 1] = c + 1 < valid ? v.y * sc : -CUDART_INF_F;
-        p[i + 2] = c + 2 < valid ? v.z * sc : -CUDART_INF_F;
-        p[i + 3] = c + 3 < valid ? v.w * sc : -CUDART_INF_F;
-        mx = fmaxf(fmaxf(mx, fmaxf(p[i], p[i + 1])), fmaxf(p[i + 2], p[i + 3]));
+      for (int q = 1; q < 4; ++q) {
+        const float4 w = *reinterpret_cast<const float4*>(sS + (q * M + srow) * kSPad + sk0);
+        v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w;
       }
+      v.x = valid > 0 ? v.x * sc : -CUDART_INF_F;
+      v.y = valid > 1 ? v.y * sc : -CUDART_INF_F;
+      v.z = valid > 2 ? v.z * sc : -CUDART_INF_F;
+      v.w = valid > 3 ? v.w * sc : -CUDART_INF_F;
+      float mx = fmaxf(fmaxf(v.x, v.y), fmaxf(v.z, v.w));
 #pragma unroll
       for (int w = 1; w < TPR; w <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, w));
       const float m_new = fmaxf(m_run, mx);
       const float ref = m_new == -CUDART_INF_F ? 0.f : m_new;
       const float alpha = fast_exp2(m_run - ref);   // 0 at the row's first tile
-      float sum = 0.f;
-#pragma unroll
-      for (int i = 0; i < KPT; ++i) { p[i] = fast_exp2(p[i] - ref); sum += p[i]; }
+      v.x = fast_exp2(v.x - ref); v.y = fast_exp2(v.y - ref); v.z = fast_exp2(v.z - ref); v.w = fast_exp2(v.w - ref);
+      float sum = (v.x + v.y) + (v.z + v.w);
 #pragma unroll
       for (int w = 1; w < TPR; w <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, w);
       l_run = l_run * alpha + sum;
       m_run = m_new;
-#pragma unroll
-      for (int i = 0; i < KPT; i += 4) {
-        const int c = sk0 + i * TPR;
-        const uint32_t addr = sP + (uint32_t)((srow * 8 + ((c >> 3) ^ (srow & 7))) * 16 + (c & 7) * 2);
-        asm volatile("st.shared.v2.b32 [%0], {%1,%2};" ::"r"(addr), "r"(pack_bf162(p[i], p[i + 1])), "r"(pack_bf162(p[i + 2], p[i + 3]))
-                     : "memory");
-      }
+      const uint32_t addr = sP + (uint32_t)((srow * 8 + ((sk0 >> 3) ^ (srow & 7))) * 16 + (sk0 & 7) * 2);
+      asm volatile("st.shared.v2.b32 [%0], {%1,%2};" ::"r"(addr), "r"(pack_bf162(v.x, v.y)), "r"(pack_bf162(v.z, v.w)) : "memory");
       if (tid % TPR == 0) { sAlpha[srow] = alpha; sL[srow] = l_run; }
     }
     __syncthreads();
@@ -310,7 +291,7 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
         const float a0 = sAlpha[m * 16 + g], a1 = sAlpha[m * 16 + g + 8];
         if (__any_sync(0xffffffffu, a0 != 1.f || a1 != 1.f)) {
 #pragma unroll
-          for (int n = 0; n < KS; ++n) { o[m][n][0] *= a0; o[m][n][1] *= a0; o[m][n][2] *= a1; o[m][n][3] *= a1; }
+          for (int n = 0; n < NT; ++n) { o[m][n][0] *= a0; o[m][n][1] *= a0; o[m][n][2] *= a1; o[m][n][3] *= a1; }
         }
       }
 #pragma unroll
@@ -324,10 +305,10 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
             ldmatrix_x4(pf[m][k], sP + (uint32_t)((r * 8 + (c8 ^ (r & 7))) * 16));
           }
 #pragma unroll
-        for (int n = 0; n < KS; ++n) {
-          if ((warp * KS + n) * 8 < R) {
+        for (int n = 0; n < NT; ++n) {
+          if ((n * 16 + warp) * 8 < R) {
             uint32_t b[4];
-            ldmatrix_x4_trans(b, sKV + stage * STAGE + key_off(k2 * 32 + lane, warp * KS + n));
+            ldmatrix_x4_trans(b, sKV + stage * STAGE + v_base + n * 2 * kSlab + k2 * 32 * 128);
 #pragma unroll
             for (int m = 0; m < MB; ++m) {
               mma_bf16_16816(o[m][n], pf[m][0], b[0], b[1]);
@@ -342,7 +323,7 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
     if (row_end || u + 1 == u1) {
       const bool whole = row_end && piece_tile0 == 0;
       const int which = cur.row == first_row ? 0 : 1;
-      if (!whole && tid % TPR == 0 && h0 + srow < a.heads) {
+      if (!whole && tid % TPR == 0 && srow < M && h0 + srow < a.heads) {
         float* ml = a.part_ml + (((long long)cta * 2 + which) * a.heads + h0 + srow) * 2;
         ml[0] = m_run;
         ml[1] = l_run;
@@ -360,8 +341,8 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
               if (a.gate != nullptr) f *= sigmoid_f(to_f(static_cast<const bf16*>(a.gate)[(long long)cur.row * a.gate_stride + head]));
             }
 #pragma unroll
-            for (int n = 0; n < KS; ++n) {
-              const int c = (warp * KS + n) * 8 + t4 * 2;
+            for (int n = 0; n < NT; ++n) {
+              const int c = (n * 16 + warp) * 8 + t4 * 2;
               if (c < R) {
                 const float x = o[m][n][2 * h] * f, y = o[m][n][2 * h + 1] * f;
                 if (whole)
@@ -429,7 +410,7 @@ __global__ void __launch_bounds__(128) latent_decode_merge_kernel(const LatentAt
 template <int KS, int MB>
 cudaError_t launch_t(const LatentAttentionArgs& a, const CUtensorMap& map, cudaStream_t s) {
   constexpr int M = 16 * MB;
-  constexpr int smem = 1024 + 2 * KS * kSlab + score_bytes(KS, MB) + M * KT * 2 + 2 * M * 4 + 12 * 4 + 2 * 8;
+  constexpr int smem = 1024 + 2 * KS * kSlab + 4 * M * kSPad * 4 + M * KS * 128 + M * KT * 2 + 2 * M * 4 + (kWarps + 2) * 4 + 2 * 8;
   static_assert(smem <= 227 * 1024, "shared memory plan exceeds the SM");
   cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<KS, MB>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (e != cudaSuccess) return e;

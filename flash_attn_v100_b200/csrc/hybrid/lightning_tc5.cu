@@ -35,19 +35,18 @@ __device__ __forceinline__ uint32_t tile_off(int row, int u) {
 __device__ __forceinline__ void st_shared(uint32_t addr, const uint4& v) {
   asm volatile("st.shared.v4.b32 [%0], {%1,%2,%3,%4};" ::"r"(addr), "r"(v.x), "r"(v.y), "r"(v.z), "r"(v.w) : "memory");
 }
-// SiLU with the hardware's exponential and reciprocal: both errors are far below the bfloat16 rounding that follows.
-__device__ __forceinline__ float silu_fast(float z) {
-  float e, r;
-  e = fast_exp2(-1.4426950408889634f * z);
-  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + e));
-  return z * r;
-}
 __device__ __forceinline__ float2 unpack2(uint32_t v) {
   return make_float2(__uint_as_float(v << 16), __uint_as_float(v & 0xffff0000u));
 }
+// SiLU of a pair with the hardware's exponential and ONE reciprocal, 1 / (ab) (the special function unit is what the activation
+// waits for); all errors are far below the bfloat16 rounding that follows.  Below -40 the sigmoid stays at its value there,
+// 4e-18, which keeps the product finite.
 __device__ __forceinline__ uint32_t silu2(uint32_t raw) {
-  const float2 f = unpack2(raw);
-  return pack_bf162(silu_fast(f.x), silu_fast(f.y));
+  const float2 z = unpack2(raw);
+  const float a = 1.f + fast_exp2(-1.4426950408889634f * fmaxf(z.x, -40.f)), b = 1.f + fast_exp2(-1.4426950408889634f * fmaxf(z.y, -40.f));
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(a * b));
+  return pack_bf162(z.x * (r * b), z.y * (r * a));
 }
 __device__ __forceinline__ uint4 silu8(const uint4& raw) {
   return make_uint4(silu2(raw.x), silu2(raw.y), silu2(raw.z), silu2(raw.w));
@@ -126,9 +125,11 @@ __global__ void __launch_bounds__(kThreads, 1) lightning_tc5_kernel(const Lightn
       else if (a.starts[seq] != 0) init = cache;
     }
 #pragma unroll
-    for (int i = 0; i < 32; ++i) {
+    for (int i = 0; i < 32; i += 4) {
       const int c = c0 + cg * 32 + i;
-      S[i] = (init != nullptr && row < a.dk && c < a.dv) ? init[(long long)row * a.dv + c] : 0.f;
+      const float4 v = init != nullptr && row < a.dk && c < a.dv ? *reinterpret_cast<const float4*>(init + (long long)row * a.dv + c)
+                                                                : make_float4(0.f, 0.f, 0.f, 0.f);
+      S[i] = v.x; S[i + 1] = v.y; S[i + 2] = v.z; S[i + 3] = v.w;
     }
   }
 
@@ -151,12 +152,26 @@ __global__ void __launch_bounds__(kThreads, 1) lightning_tc5_kernel(const Lightn
     }
   };
 
+  // The finished chunk's output lies in the Q tile; every thread stores the units it will overwrite with the next queries.
+  auto store_out = [&](int done) {
+    const long long tb = t0 + (long long)done * C + urow;
+    bf16* p = static_cast<bf16*>(a.out) + tb * ((long long)a.heads * a.dv) + (long long)head * a.dv + c0 + cu8;
+#pragma unroll
+    for (int n = 0; n < 4; ++n) {
+      uint4 v;
+      asm volatile("ld.shared.v4.b32 {%0,%1,%2,%3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w)
+                   : "r"(sQ + tile_off(urow + 32 * n, tid & 15)) : "memory");
+      if (v_ok && tb + 32 * n < t1) *reinterpret_cast<uint4*>(p + (long long)(32 * n) * a.heads * a.dv) = v;
+    }
+  };
+
   bool ok = true;
   uint32_t phase = 0;
   fetch(0);
   int chunk = 0;
   for (; chunk < n_chunk; ++chunk, phase ^= 1u) {
     const int rows = min(C, n_tok - chunk * C);
+    if (!STATE_ONLY && chunk > 0) store_out(chunk - 1);
     // ---- activated tiles, decayed keys, state -------------------------------------------------------
 #pragma unroll
     for (int n = 0; n < 4; ++n) {
@@ -275,23 +290,19 @@ __global__ void __launch_bounds__(kThreads, 1) lightning_tc5_kernel(const Lightn
       ok = mbar_wait(bar_o, phase) && ok;
       tc_fence_after();
       const float w = pw[min(row + 1, C)];
-      bf16* orow = static_cast<bf16*>(a.out) + (t0 + (long long)chunk * C + row) * ((long long)a.heads * a.dv) + (long long)head * a.dv + c0;
 #pragma unroll
       for (int h = 0; h < 2; ++h) {
         float x[16], y[16];
         tc_ld16(tO1 + h * 16u, x);
         tc_ld16(tO2 + h * 16u, y);
         tc_wait_ld();
-        if (row < rows) {
 #pragma unroll
-          for (int u = 0; u < 2; ++u) {
-            const int c = cg * 32 + h * 16 + u * 8;
-            uint32_t p[4];
+        for (int u = 0; u < 2; ++u) {
+          uint32_t p[4];
 #pragma unroll
-            for (int i = 0; i < 4; ++i)
-              p[i] = pack_bf162(w * x[u * 8 + 2 * i] + y[u * 8 + 2 * i], w * x[u * 8 + 2 * i + 1] + y[u * 8 + 2 * i + 1]);
-            if (c0 + c < a.dv) *reinterpret_cast<uint4*>(orow + c) = make_uint4(p[0], p[1], p[2], p[3]);
-          }
+          for (int i = 0; i < 4; ++i)
+            p[i] = pack_bf162(w * x[u * 8 + 2 * i] + y[u * 8 + 2 * i], w * x[u * 8 + 2 * i + 1] + y[u * 8 + 2 * i + 1]);
+          st_shared(sQ + tile_off(row, cg * 4 + h * 2 + u), make_uint4(p[0], p[1], p[2], p[3]));   // Q is no longer read
         }
       }
     }
@@ -305,12 +316,13 @@ __global__ void __launch_bounds__(kThreads, 1) lightning_tc5_kernel(const Lightn
     }
     mbar_wait(bar_s, phase);
   }
+  if (!STATE_ONLY && chunk == n_chunk) store_out(n_chunk - 1);
   float* dst = STATE_ONLY ? segst : (last_seg ? cache : nullptr);
   if (dst != nullptr && row < a.dk) {
 #pragma unroll
-    for (int i = 0; i < 32; ++i) {
+    for (int i = 0; i < 32; i += 4) {
       const int c = c0 + cg * 32 + i;
-      if (c < a.dv) dst[(long long)row * a.dv + c] = S[i];
+      if (c < a.dv) *reinterpret_cast<float4*>(dst + (long long)row * a.dv + c) = make_float4(S[i], S[i + 1], S[i + 2], S[i + 3]);
     }
   }
   tc_fence_before();
