@@ -7,8 +7,8 @@
 //
 // Sixteen warps.  Scores: warp = (a quarter of the tile's keys) x (one 16-column step of every slab); the four partial score
 // tiles are added up in shared memory by the softmax.  Values: warp = 8 columns of
-// every other slab.  (With these shares every shared-memory address is a per-warp base plus a constant.)  Warp 0 fetches the next tile by TMA (one box of 16 rows x 64 columns per page and slab, 128-byte swizzle)
-// while the current one is computed.  The wait for a tile is bounded; one that runs out sets the status word.
+// every other slab.  (With these shares every shared-memory address is a per-warp base plus a constant.)  The next tile is fetched by TMA while the current one is computed: one box of 16 rows x 64 columns per page
+// and slab (128-byte swizzle), the boxes spread over all warps so that none of them falls behind.  The wait for a tile is bounded; one that runs out sets the status word.
 #include <math_constants.h>
 
 #include "../common.cuh"
@@ -115,8 +115,8 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
   }
   const int first_row = found[0];
   if (tid == 0) {
-    mbar_init(bars, 1);
-    mbar_init(bars + 8, 1);
+    mbar_init(bars, 4 * KS);                        // one arrival per box
+    mbar_init(bars + 8, 4 * KS);
     mbar_fence_init();
     fence_proxy_async();
     tma_prefetch_desc(&pool_map);
@@ -128,30 +128,24 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
     if (++c.tile == c.tiles && c.row + 1 < a.rows) start_row(c, c.row + 1);
   };
 
-  // ---- copies (warp 0) ----------------------------------------------------------------------------
+  // ---- copies: lane l of warp w fetches box l * kWarps + w of a tile --------------------------------
   bool bad = false, late = false;
-  // lanes 0-3: pages of the cursor's tile (-1: no keys there, -2: not a page of a request); checked when they are used
-  auto tile_pages = [&](const Cursor& c) {
-    const int seq = a.tok_seq[c.row], key = c.tile * KT + lane * 16;
-    if (lane >= 4 || (key >= c.n && lane > 0)) return -1;
-    if (seq < 0 || seq >= a.n_seq || c.n <= 0 || (key >> 4) >= a.max_blocks) return -2;
-    return a.block_table[(long long)seq * a.max_blocks + (key >> 4)];
+  const int box = lane * kWarps + warp, quarter = box / KS, slab = box - quarter * KS;
+  const bool fetcher = box < 4 * KS;
+  // page of the cursor's tile that my box comes from, checked when it is used; keys past the end: the tile's first page (any
+  // finite rows will do, their weights are zero)
+  auto box_page = [&](const Cursor& c) {
+    if (!fetcher) return 0;
+    const int seq = a.tok_seq[c.row];
+    int blk = c.tile * (KT / 16) + quarter;
+    if (blk * 16 >= c.n) blk = c.tile * (KT / 16);
+    return seq >= 0 && seq < a.n_seq && c.n > 0 && blk < a.max_blocks ? a.block_table[(long long)seq * a.max_blocks + blk] : -1;
   };
-  auto copy_tile = [&](int page, int stage) {
-    const bool wrong = lane < 4 && page != -1 && (page < 0 || page >= a.n_blocks);
-    bad |= wrong;
-    if (wrong) page = 0;
-    const int p0 = __shfl_sync(0xffffffffu, page, 0);
-    if (page < 0) page = p0;                        // keys past the end: any page, their weights are zero
-    if (lane == 0) mbar_expect_tx(bars + 8 * stage, STAGE);
-    __syncwarp();
-#pragma unroll
-    for (int b = 0; b < 4 * KS; b += 32) {
-      const int i = b + lane, slab = i % KS, quarter = i / KS;
-      const int pg = __shfl_sync(0xffffffffu, page, quarter & 3);
-      if (i < 4 * KS)
-        tma_load_2d_nohint(sKV + stage * STAGE + slab * kSlab + quarter * 2048, &pool_map, slab * 64, pg * 16, bars + 8 * stage);
-    }
+  auto copy_box = [&](int page, int stage) {
+    if (!fetcher) return;
+    if (page < 0 || page >= a.n_blocks) { bad = true; page = 0; }
+    mbar_expect_tx(bars + 8 * stage, 2048);
+    tma_load_2d_nohint(sKV + stage * STAGE + slab * kSlab + quarter * 2048, &pool_map, slab * 64, page * 16, bars + 8 * stage);
   };
 
   // ---- per-row state ----------------------------------------------------------------------------
@@ -200,13 +194,11 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
   cur.tile = u0 - found[1];
   Cursor nxt = cur;
   int piece_tile0 = cur.tile;
-  int page_next = -1;
-  if (warp == 0) {
-    copy_tile(tile_pages(nxt), 0);
-    if (u0 + 1 < u1) {
-      advance(nxt);
-      page_next = tile_pages(nxt);
-    }
+  int page_next = 0;
+  copy_box(box_page(nxt), 0);
+  if (u0 + 1 < u1) {
+    advance(nxt);
+    page_next = box_page(nxt);
   }
   load_q(cur.row);
 
@@ -214,11 +206,11 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
   for (int u = u0; u < u1; ++u) {
     const int stage = (u - u0) & 1;
     __syncthreads();                                // the other stage and the score tiles are no longer read
-    if (warp == 0 && u + 1 < u1) {
-      copy_tile(page_next, stage ^ 1);
+    if (u + 1 < u1) {
+      copy_box(page_next, stage ^ 1);
       if (u + 2 < u1) {
         advance(nxt);
-        page_next = tile_pages(nxt);
+        page_next = box_page(nxt);
       }
     }
     if (!late) late = !mbar_wait(bars + 8 * stage, (uint32_t)((u - u0) >> 1) & 1u);

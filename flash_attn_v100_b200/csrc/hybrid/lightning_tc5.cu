@@ -25,7 +25,7 @@ constexpr int N = 128;         // key and value columns per CTA (padded with zer
 constexpr int kThreads = 512;
 constexpr int SLAB = 128 * 128;
 constexpr int TILE = 2 * SLAB;
-constexpr int kSmem = 1024 + 7 * TILE + (C + 1) * 4 + 12 + 4 * 8 + 16;
+constexpr int kSmem = 1024 + 7 * TILE + (2 * C + 4) * 4 + 4 * 8 + 16;
 static_assert(kSmem <= 227 * 1024, "shared memory plan exceeds the SM");
 
 // Byte offset of 16-byte unit `u` (0..15) of row `row` in a tile.
@@ -67,8 +67,9 @@ __global__ void __launch_bounds__(kThreads, 1) lightning_tc5_kernel(const Lightn
   const uint32_t raw_base = smem_u32(smem_dyn);
   uint8_t* smem = smem_dyn + ((1024u - (raw_base & 1023u)) & 1023u);
   const uint32_t sQ = smem_u32(smem), sK = sQ + TILE, sV = sK + TILE, sKh = sV + TILE, sKl = sKh + TILE, sSh = sKl + TILE, sSl = sSh + TILE;
-  float* pw = reinterpret_cast<float*>(smem + 7 * TILE);               // decay^0 .. decay^C
-  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + 7 * TILE + ((C + 1) * 4 + 12) / 16 * 16);
+  float* pz = reinterpret_cast<float*>(smem + 7 * TILE);               // [C] zeros, the weights of later tokens, then
+  float* pw = pz + C;                                                  // decay^0 .. decay^C
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + 7 * TILE + (2 * C + 4) * 4);
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 4);
   const uint32_t bar_a = smem_u32(bars), bar_s = smem_u32(bars + 1), bar_o = smem_u32(bars + 2);
 
@@ -103,7 +104,10 @@ __global__ void __launch_bounds__(kThreads, 1) lightning_tc5_kernel(const Lightn
   }
   {
     const float d = a.decay[head];
-    for (int i = tid; i <= C; i += kThreads) pw[i] = i == 0 ? 1.f : powf(d, (float)i);
+    for (int i = tid; i <= C; i += kThreads) {
+      pw[i] = i == 0 ? 1.f : powf(d, (float)i);
+      if (i < C) pz[i] = 0.f;
+    }
   }
   tc_fence_before();
   __syncthreads();
@@ -165,12 +169,27 @@ __global__ void __launch_bounds__(kThreads, 1) lightning_tc5_kernel(const Lightn
     }
   };
 
+  // the rows that fetch() will read, on their way to the L2 while the current chunk is computed
+  auto prefetch = [&](int chunk) {
+    const long long tb = t0 + (long long)chunk * C + urow;
+#pragma unroll
+    for (int n = 0; n < 4; ++n) {
+      if (tb + 32 * n < t1 && (tid & 7) == 0) {
+        const bf16* pr = base + (tb + 32 * n) * a.stride;
+        if (!STATE_ONLY && k_ok) asm volatile("prefetch.global.L2 [%0];" ::"l"(pr + a.off_q + head * a.dk + cu8));
+        if (k_ok) asm volatile("prefetch.global.L2 [%0];" ::"l"(pr + a.off_k + head * a.dk + cu8));
+        if (v_ok) asm volatile("prefetch.global.L2 [%0];" ::"l"(pr + a.off_v + head * a.dv + c0 + cu8));
+      }
+    }
+  };
+
   bool ok = true;
   uint32_t phase = 0;
   fetch(0);
   int chunk = 0;
   for (; chunk < n_chunk; ++chunk, phase ^= 1u) {
     const int rows = min(C, n_tok - chunk * C);
+    if (chunk + 1 < n_chunk) prefetch(chunk + 1);
     if (!STATE_ONLY && chunk > 0) store_out(chunk - 1);
     // ---- activated tiles, decayed keys, state -------------------------------------------------------
 #pragma unroll
@@ -244,15 +263,14 @@ __global__ void __launch_bounds__(kThreads, 1) lightning_tc5_kernel(const Lightn
       tc_fence_before();
       __syncthreads();                                        // P is written over other warps' part of A
       tc_fence_after();
-      const float* pr = pw + (row - cg * 32);
-      const int lim = row - cg * 32;                          // my columns 0 .. lim are at or before my row
+      const float* pr = pw + (row - cg * 32);                 // pr[-j]: weight of my column j (0 past my row)
 #pragma unroll
       for (int h = 0; h < 2; ++h) {
         uint32_t ph[8], pl[8];
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
           const int j = h * 16 + 2 * i;
-          const float x = j <= lim ? s[j] * pr[-j] : 0.f, y = j + 1 <= lim ? s[j + 1] * pr[-j - 1] : 0.f;
+          const float x = s[j] * pr[-j], y = s[j + 1] * pr[-j - 1];
           split2(x, y, ph[i], pl[i]);
         }
         tc_st8(tP + h * 8u, ph);
