@@ -5,10 +5,11 @@
 // 32, the M rows of the MMAs) as key and as value.  The (row, key tile) units of the batch are numbered row by row and cut
 // into equal runs, one per CTA, whatever the lengths; a row that is cut leaves partial sums that a second kernel merges.
 //
-// Sixteen warps.  Scores: warp = (a quarter of the tile's keys) x (one 16-column step of every slab); the four partial score
-// tiles are added up in shared memory by the softmax.  Values: warp = 8 columns of
-// every other slab.  (With these shares every shared-memory address is a per-warp base plus a constant.)  The next tile is fetched by TMA while the current one is computed: one box of 16 rows x 64 columns per page
-// and slab (128-byte swizzle), the boxes spread over all warps so that none of them falls behind.  The wait for a tile is bounded; one that runs out sets the status word.
+// Sixteen warps compute.  Scores: warp = (a quarter of the tile's keys) x (one 16-column step of every slab); the four partial
+// score tiles are added up in shared memory by the softmax.  Values: warp = 8 columns of every other slab.  (With these shares
+// every shared-memory address is a per-warp base plus a constant.)  A seventeenth warp fetches the tiles by TMA, one box of 16
+// rows x 64 columns per page and slab (128-byte swizzle), one tile ahead.  Waits are bounded; one that runs out sets the status
+// word.
 #include <math_constants.h>
 
 #include "../common.cuh"
@@ -24,7 +25,8 @@ typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t,
                                   CUtensorMapFloatOOBfill);
 
 constexpr int KT = 64;         // keys per tile
-constexpr int kThreads = 512;
+constexpr int kCompute = 512;  // threads that compute
+constexpr int kThreads = kCompute + 32;
 constexpr int kWarps = kThreads / 32;
 constexpr int kSPad = KT + 8;  // row stride of the partial score tiles
 constexpr int kSlab = KT * 128;
@@ -80,27 +82,30 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
   float* sL = sAlpha + M;                                          // [M]
   int* scan_buf = reinterpret_cast<int*>(sL + M);                  // [kWarps]
   int* found = scan_buf + kWarps;                                  // [2] first row, its first unit
-  const uint32_t bars = smem_u32(scan_buf + kWarps + 2);           // [2] tile has landed
+  const uint32_t bars = smem_u32(scan_buf + kWarps + 3);           // [2] tile has landed, [2] tile is no longer read
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
   const int cta = blockIdx.x, h0 = blockIdx.y * M;
   const int R = a.kv_rank, D = R + a.rot_dim;
 
   // ---- my run of units --------------------------------------------------------------------------
-  int total = 0;
+  int total = 0, mine = 0, upto = 0;               // of my row in the last block of rows: its tiles, tiles up to and with it
   for (long long r0 = 0; r0 < a.rows; r0 += kThreads) {
-    const int v = r0 + tid < a.rows ? row_tiles_of(a, r0 + tid) : 0;
-    const int inc = block_scan(v, scan_buf);
-    if (cta == 0 && blockIdx.y == 0 && r0 + tid < a.rows) a.row_tiles[r0 + tid + 1] = total + inc;
-    if (tid == kThreads - 1) found[0] = inc;
+    mine = r0 + tid < a.rows ? row_tiles_of(a, r0 + tid) : 0;
+    upto = total + block_scan(mine, scan_buf);
+    if (cta == 0 && blockIdx.y == 0 && r0 + tid < a.rows) a.row_tiles[r0 + tid + 1] = upto;
+    if (tid == kThreads - 1) found[0] = upto;
     __syncthreads();
-    total += found[0];
+    total = found[0];
     __syncthreads();
   }
   if (cta == 0 && blockIdx.y == 0 && tid == 0) a.row_tiles[0] = 0;
   const int per = (total + a.n_cta - 1) / a.n_cta;
   const int u0 = cta * per, u1 = min(u0 + per, total);
   if (u0 >= u1) return;
-  {
+  if (a.rows <= kThreads) {
+    if (mine > 0 && upto - mine <= u0 && u0 < upto) { found[0] = tid; found[1] = upto - mine; }
+    __syncthreads();
+  } else {
     int base = 0;
     for (long long r0 = 0; r0 < a.rows; r0 += kThreads) {
       const int v = r0 + tid < a.rows ? row_tiles_of(a, r0 + tid) : 0;
@@ -117,6 +122,8 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
   if (tid == 0) {
     mbar_init(bars, 4 * KS);                        // one arrival per box
     mbar_init(bars + 8, 4 * KS);
+    mbar_init(bars + 16, kCompute / 32);            // one arrival per computing warp
+    mbar_init(bars + 24, kCompute / 32);
     mbar_fence_init();
     fence_proxy_async();
     tma_prefetch_desc(&pool_map);
@@ -128,25 +135,58 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
     if (++c.tile == c.tiles && c.row + 1 < a.rows) start_row(c, c.row + 1);
   };
 
-  // ---- copies: lane l of warp w fetches box l * kWarps + w of a tile --------------------------------
-  bool bad = false, late = false;
-  const int box = lane * kWarps + warp, quarter = box / KS, slab = box - quarter * KS;
-  const bool fetcher = box < 4 * KS;
-  // page of the cursor's tile that my box comes from, checked when it is used; keys past the end: the tile's first page (any
-  // finite rows will do, their weights are zero)
-  auto box_page = [&](const Cursor& c) {
-    if (!fetcher) return 0;
-    const int seq = a.tok_seq[c.row];
-    int blk = c.tile * (KT / 16) + quarter;
-    if (blk * 16 >= c.n) blk = c.tile * (KT / 16);
-    return seq >= 0 && seq < a.n_seq && c.n > 0 && blk < a.max_blocks ? a.block_table[(long long)seq * a.max_blocks + blk] : -1;
+  bool late = false;
+  auto wait = [&](uint32_t bar, uint32_t parity) {
+    if (!late) late = !mbar_wait(bar, parity);
   };
-  auto copy_box = [&](int page, int stage) {
-    if (!fetcher) return;
-    if (page < 0 || page >= a.n_blocks) { bad = true; page = 0; }
-    mbar_expect_tx(bars + 8 * stage, 2048);
-    tma_load_2d_nohint(sKV + stage * STAGE + slab * kSlab + quarter * 2048, &pool_map, slab * 64, page * 16, bars + 8 * stage);
-  };
+
+  if (warp == kCompute / 32) {
+    // ---- copies: lane l fetches boxes l and l + 32 of every tile ------------------------------------
+    constexpr int NB = (4 * KS + 31) / 32;
+    bool bad = false;
+    // page of the cursor's tile that a box comes from, checked when it is used; keys past the end: the tile's first page (any
+    // finite rows will do, their weights are zero)
+    auto box_page = [&](const Cursor& c, int box) {
+      const int seq = a.tok_seq[c.row];
+      int blk = c.tile * (KT / 16) + box / KS;
+      if (blk * 16 >= c.n) blk = c.tile * (KT / 16);
+      return seq >= 0 && seq < a.n_seq && c.n > 0 && blk < a.max_blocks ? a.block_table[(long long)seq * a.max_blocks + blk] : -1;
+    };
+    Cursor nxt;
+    start_row(nxt, first_row);
+    nxt.tile = u0 - found[1];
+    int page[NB];
+#pragma unroll
+    for (int i = 0; i < NB; ++i) page[i] = lane + 32 * i < 4 * KS ? box_page(nxt, lane + 32 * i) : 0;
+#pragma unroll 1
+    for (int u = u0; u < u1; ++u) {
+      const int k = u - u0, stage = k & 1;
+      if (k >= 2) wait(bars + 16 + 8 * stage, (uint32_t)((k >> 1) - 1) & 1u);
+#pragma unroll
+      for (int i = 0; i < NB; ++i) {
+        const int box = lane + 32 * i;
+        if (box < 4 * KS) {
+          if (page[i] < 0 || page[i] >= a.n_blocks) { bad = true; page[i] = 0; }
+          mbar_expect_tx(bars + 8 * stage, 2048);
+          tma_load_2d_nohint(sKV + stage * STAGE + (box % KS) * kSlab + (box / KS) * 2048, &pool_map, (box % KS) * 64, page[i] * 16,
+                             bars + 8 * stage);
+        }
+      }
+      if (u + 1 < u1) {
+        advance(nxt);
+#pragma unroll
+        for (int i = 0; i < NB; ++i)
+          if (lane + 32 * i < 4 * KS) page[i] = box_page(nxt, lane + 32 * i);
+      }
+    }
+    // leave only when every copy has landed
+    for (int k = u1 - u0 >= 2 ? u1 - u0 - 2 : 0; k < u1 - u0; ++k)
+      if (!mbar_wait(bars + 8 * (k & 1), (uint32_t)(k >> 1) & 1u)) late = true;
+    if (bad) atomicOr(a.status, kStatusBadPageId);
+    if (late) atomicOr(a.status, kStatusWaitTimeout);
+    return;
+  }
+  auto sync = [&]() { asm volatile("bar.sync 1, %0;" ::"n"(kCompute) : "memory"); };
 
   // ---- per-row state ----------------------------------------------------------------------------
   const int slice = warp & 3, kquarter = warp >> 2;
@@ -158,7 +198,7 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
   auto load_q = [&](long long row) {
     const int half = a.rot_dim / 2;
 #pragma unroll 1
-    for (int idx = tid; idx < M * UNITS; idx += kThreads) {
+    for (int idx = tid; idx < M * UNITS; idx += kCompute) {
       const int m = idx / UNITS, u = idx - m * UNITS, c = u * 8, head = h0 + m;
       uint4 v = make_uint4(0, 0, 0, 0);
       if (head < a.heads) {
@@ -192,28 +232,14 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
   Cursor cur;
   start_row(cur, first_row);
   cur.tile = u0 - found[1];
-  Cursor nxt = cur;
   int piece_tile0 = cur.tile;
-  int page_next = 0;
-  copy_box(box_page(nxt), 0);
-  if (u0 + 1 < u1) {
-    advance(nxt);
-    page_next = box_page(nxt);
-  }
   load_q(cur.row);
+  sync();
 
 #pragma unroll 1
   for (int u = u0; u < u1; ++u) {
     const int stage = (u - u0) & 1;
-    __syncthreads();                                // the other stage and the score tiles are no longer read
-    if (u + 1 < u1) {
-      copy_box(page_next, stage ^ 1);
-      if (u + 2 < u1) {
-        advance(nxt);
-        page_next = box_page(nxt);
-      }
-    }
-    if (!late) late = !mbar_wait(bars + 8 * stage, (uint32_t)((u - u0) >> 1) & 1u);
+    wait(bars + 8 * stage, (uint32_t)((u - u0) >> 1) & 1u);
     // ---- partial scores -------------------------------------------------------------------------
     {
       float s[MB][2][4];
@@ -245,7 +271,7 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
             *reinterpret_cast<float2*>(sS + (slice * M + m * 16 + g + h * 8) * kSPad + kquarter * 16 + n * 8 + t4 * 2) =
                 make_float2(s[m][n][2 * h], s[m][n][2 * h + 1]);
     }
-    __syncthreads();
+    sync();
     // ---- softmax of my row's keys ---------------------------------------------------------------
     if (srow < M) {                                 // (whole warps)
       const int valid = cur.n - cur.tile * KT - sk0;
@@ -275,7 +301,7 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
       asm volatile("st.shared.v2.b32 [%0], {%1,%2};" ::"r"(addr), "r"(pack_bf162(v.x, v.y)), "r"(pack_bf162(v.z, v.w)) : "memory");
       if (tid % TPR == 0) { sAlpha[srow] = alpha; sL[srow] = l_run; }
     }
-    __syncthreads();
+    sync();
     // ---- values: my columns of the latents --------------------------------------------------------
     {
 #pragma unroll
@@ -310,6 +336,8 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
         }
       }
     }
+    __syncwarp();
+    if (lane == 0) mbar_arrive(bars + 16 + 8 * stage);
     // ---- end of a row or of my run ------------------------------------------------------------------
     const bool row_end = cur.tile + 1 == cur.tiles;
     if (row_end || u + 1 == u1) {
@@ -349,49 +377,52 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
         m_run = -CUDART_INF_F;
         l_run = 0.f;
         load_q(cur.row + 1);
+        sync();
         piece_tile0 = 0;
       }
     }
     if (u + 1 < u1) advance(cur);
   }
-  if (bad) atomicOr(a.status, kStatusBadPageId);
-  if (late) {                                       // leave only after another (bounded) wait for the copies in flight
-    atomicOr(a.status, kStatusWaitTimeout);
-    for (int i = u1 - u0 >= 2 ? u1 - 2 : u1 - 1; i < u1; ++i) mbar_wait(bars + 8 * ((i - u0) & 1), (uint32_t)((i - u0) >> 1) & 1u);
-  }
+  if (late && lane == 0) atomicOr(a.status, kStatusWaitTimeout);
 }
 
 // Rows that several CTAs worked on: log-sum-exp merge of their partial sums.  One CTA per (row, head).
-__global__ void __launch_bounds__(128) latent_decode_merge_kernel(const LatentAttentionArgs a) {
+constexpr int kMergeThreads = 128;
+__global__ void __launch_bounds__(kMergeThreads) latent_decode_merge_kernel(const LatentAttentionArgs a) {
+  extern __shared__ float weight[];                 // [pieces of the row] (n_cta at most)
+  __shared__ float red[2 * kMergeThreads / 32];
   const long long row = blockIdx.x;
-  const int head = blockIdx.y;
+  const int head = blockIdx.y, tid = threadIdx.x;
   const int b0 = a.row_tiles[row], b1 = a.row_tiles[row + 1], total = a.row_tiles[a.rows];
   const int per = (total + a.n_cta - 1) / a.n_cta;
-  const int c0 = b0 / per, c1 = (b1 - 1) / per;
-  if (c0 == c1) return;                             // one CTA had the whole row
-  // the row is CTA c's first one exactly if the CTA's run starts inside it or at its first unit
+  const int c0 = b0 / per, n = (b1 - 1) / per - c0 + 1;
+  if (n == 1) return;                               // one CTA had the whole row
+  // the row is a CTA's first one exactly if the CTA's run starts inside it or at its first unit
+  auto piece = [&](int i) { return ((long long)(c0 + i) * 2 + ((c0 + i) * per >= b0 ? 0 : 1)) * a.heads + head; };
   float m = -CUDART_INF_F;
-  for (int c = c0; c <= c1; ++c) {
-    const int which = c * per >= b0 ? 0 : 1;
-    m = fmaxf(m, a.part_ml[(((long long)c * 2 + which) * a.heads + head) * 2]);
-  }
+  for (int i = tid; i < n; i += kMergeThreads) m = fmaxf(m, a.part_ml[piece(i) * 2]);
+  m = warp_max(m);
+  if ((tid & 31) == 0) red[tid >> 5] = m;
+  __syncthreads();
+  m = fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3]));
   float l = 0.f;
-  for (int c = c0; c <= c1; ++c) {
-    const float* ml = a.part_ml + (((long long)c * 2 + (c * per >= b0 ? 0 : 1)) * a.heads + head) * 2;
-    l += ml[1] * exp2f(ml[0] - m);
+  for (int i = tid; i < n; i += kMergeThreads) {
+    const float w = exp2f(a.part_ml[piece(i) * 2] - m);
+    weight[i] = w;
+    l += w * a.part_ml[piece(i) * 2 + 1];
   }
+  l = block_sum(l, red + 4);
   float f = l > 0.f ? 1.f / l : 0.f;
   if (a.gate != nullptr) f *= sigmoid_f(to_f(static_cast<const bf16*>(a.gate)[row * a.gate_stride + head]));
   bf16* out = static_cast<bf16*>(a.out) + (row * a.heads + head) * a.kv_rank;
-  for (int i = threadIdx.x * 4; i < a.kv_rank; i += 128 * 4) {
+  for (int i = tid * 4; i < a.kv_rank; i += kMergeThreads * 4) {
     float acc[4] = {0.f, 0.f, 0.f, 0.f};
-    for (int c = c0; c <= c1; ++c) {
-      const long long s = ((long long)c * 2 + (c * per >= b0 ? 0 : 1)) * a.heads + head;
-      const float w = exp2f(a.part_ml[s * 2] - m);
+#pragma unroll 8
+    for (int c = 0; c < n; ++c) {
       float v[4];
-      load_n<4>(a.part_o + s * a.kv_rank + i, v);
+      load_n<4>(a.part_o + piece(c) * a.kv_rank + i, v);
 #pragma unroll
-      for (int j = 0; j < 4; ++j) acc[j] += w * v[j];
+      for (int j = 0; j < 4; ++j) acc[j] += weight[c] * v[j];
     }
 #pragma unroll
     for (int j = 0; j < 4; ++j) acc[j] *= f;
@@ -402,12 +433,12 @@ __global__ void __launch_bounds__(128) latent_decode_merge_kernel(const LatentAt
 template <int KS, int MB>
 cudaError_t launch_t(const LatentAttentionArgs& a, const CUtensorMap& map, cudaStream_t s) {
   constexpr int M = 16 * MB;
-  constexpr int smem = 1024 + 2 * KS * kSlab + 4 * M * kSPad * 4 + M * KS * 128 + M * KT * 2 + 2 * M * 4 + (kWarps + 2) * 4 + 2 * 8;
+  constexpr int smem = 1024 + 2 * KS * kSlab + 4 * M * kSPad * 4 + M * KS * 128 + M * KT * 2 + 2 * M * 4 + (kWarps + 3) * 4 + 4 * 8;
   static_assert(smem <= 227 * 1024, "shared memory plan exceeds the SM");
   cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<KS, MB>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (e != cudaSuccess) return e;
   latent_decode_kernel<KS, MB><<<dim3((unsigned)a.n_cta, (unsigned)((a.heads + M - 1) / M)), kThreads, smem, s>>>(map, a);
-  latent_decode_merge_kernel<<<dim3((unsigned)a.rows, (unsigned)a.heads), 128, 0, s>>>(a);
+  latent_decode_merge_kernel<<<dim3((unsigned)a.rows, (unsigned)a.heads), kMergeThreads, a.n_cta * sizeof(float), s>>>(a);
   return cudaGetLastError();
 }
 
