@@ -208,13 +208,30 @@ __global__ void __launch_bounds__(kThreads) side_gate_kernel(const T* z, const T
 }
 
 // One CTA per row: norms of the two latents, rotation of the shared key part, append of (latent, rotated part) to the
-// row's place in the paged cache.
-template <typename T>
-__global__ void __launch_bounds__(128) latent_prep_kernel(const LatentPrepArgs a) {
-  __shared__ float red[4];
+// row's place in the paged cache.  NQ / NK: vectors per thread that hold the query / key-value latent between the sum of squares
+// and the scaling (0: any size, the row is read twice).
+template <typename T, int VEC, int NQ, int NK>
+__global__ void __launch_bounds__(kThreads) latent_prep_kernel(const LatentPrepArgs a) {
+  __shared__ float red[2][kThreads / 32];
   const long long row = blockIdx.x;
+  const int tid = threadIdx.x;
   const T* in = static_cast<const T*>(a.down) + row * a.down_stride;
   const T *zq = in + a.off_q, *zk = in + a.off_kv, *zr = in + a.off_r;
+  const int nq = a.q_rank / VEC, nk = a.kv_rank / VEC, half = a.rot_dim / 2;
+  float kq[NQ > 0 ? NQ : 1][VEC], kk[NK > 0 ? NK : 1][VEC];
+  float sq = 0.f, sk = 0.f;
+  auto add = [](float& s, const float (&v)[VEC]) {
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) s += v[i] * v[i];
+  };
+  if constexpr (NQ > 0) {
+#pragma unroll
+    for (int n = 0; n < NQ; ++n)
+      if (tid + n * kThreads < nq) load_n<VEC>(zq + (tid + n * kThreads) * VEC, kq[n]);
+#pragma unroll
+    for (int n = 0; n < NK; ++n)
+      if (tid + n * kThreads < nk) load_n<VEC>(zk + (tid + n * kThreads) * VEC, kk[n]);
+  }
   T* pool_row = nullptr;
   {
     const int seq = a.tok_seq[row], pos = a.positions[row];
@@ -223,34 +240,65 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(const LatentPrepArgs a
     if (seq >= 0 && seq < a.n_seq && pos >= 0 && blk < a.max_blocks) page = a.block_table[(long long)seq * a.max_blocks + blk];
     if (page >= 0 && page < a.n_blocks) {
       pool_row = static_cast<T*>(a.pool) + ((long long)page * 16 + (pos & 15)) * a.pool_stride;
-    } else if (threadIdx.x == 0) {
+    } else if (tid == 0) {
       atomicOr(a.status, 2);
     }
   }
-  float ss = 0.f;
-  for (int c = threadIdx.x; c < a.q_rank; c += blockDim.x) { const float v = to_f(zq[c]); ss += v * v; }
-  const float qinv = 1.f / sqrtf(block_sum(ss, red) / (float)a.q_rank + a.eps);
-  T* cq = static_cast<T*>(a.cq) + row * a.q_rank;
-  const T* wq = static_cast<const T*>(a.wq);
-  for (int c = threadIdx.x; c < a.q_rank; c += blockDim.x) cq[c] = from_f<T>(to_f(zq[c]) * qinv * to_f(wq[c]));
-  ss = 0.f;
-  for (int c = threadIdx.x; c < a.kv_rank; c += blockDim.x) { const float v = to_f(zk[c]); ss += v * v; }
-  const float kinv = 1.f / sqrtf(block_sum(ss, red) / (float)a.kv_rank + a.eps);
-  const T* wkv = static_cast<const T*>(a.wkv);
-  T* c_out = a.c_out ? static_cast<T*>(a.c_out) + row * a.kv_rank : nullptr;
-  for (int c = threadIdx.x; c < a.kv_rank; c += blockDim.x) {
-    const T v = from_f<T>(to_f(zk[c]) * kinv * to_f(wkv[c]));
-    if (pool_row) pool_row[c] = v;
-    if (c_out) c_out[c] = v;
-  }
-  const int half = a.rot_dim / 2;
   T* r_out = a.r_out ? static_cast<T*>(a.r_out) + row * a.rot_dim : nullptr;
-  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+  for (int i = tid; i < half; i += kThreads) {
     const float cs = a.cos_t[row * half + i], sn = a.sin_t[row * half + i];
     const float u = to_f(zr[i]), v = to_f(zr[i + half]);
     const T ru = from_f<T>(u * cs - v * sn), rv = from_f<T>(v * cs + u * sn);
     if (pool_row) { pool_row[a.kv_rank + i] = ru; pool_row[a.kv_rank + half + i] = rv; }
     if (r_out) { r_out[i] = ru; r_out[half + i] = rv; }
+  }
+  if constexpr (NQ > 0) {
+#pragma unroll
+    for (int n = 0; n < NQ; ++n)
+      if (tid + n * kThreads < nq) add(sq, kq[n]);
+#pragma unroll
+    for (int n = 0; n < NK; ++n)
+      if (tid + n * kThreads < nk) add(sk, kk[n]);
+  } else {
+    for (int c = tid; c < nq; c += kThreads) { load_n<VEC>(zq + c * VEC, kq[0]); add(sq, kq[0]); }
+    for (int c = tid; c < nk; c += kThreads) { load_n<VEC>(zk + c * VEC, kk[0]); add(sk, kk[0]); }
+  }
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  if ((tid & 31) == 0) { red[0][tid >> 5] = sq; red[1][tid >> 5] = sk; }
+  __syncthreads();
+  sq = sk = 0.f;
+#pragma unroll
+  for (int i = 0; i < kThreads / 32; ++i) { sq += red[0][i]; sk += red[1][i]; }
+  const float qinv = 1.f / sqrtf(sq / (float)a.q_rank + a.eps), kinv = 1.f / sqrtf(sk / (float)a.kv_rank + a.eps);
+  T* cq = static_cast<T*>(a.cq) + row * a.q_rank;
+  T* c_out = a.c_out ? static_cast<T*>(a.c_out) + row * a.kv_rank : nullptr;
+  const T *wq = static_cast<const T*>(a.wq), *wkv = static_cast<const T*>(a.wkv);
+  auto scale = [](float (&v)[VEC], float inv, const T* w) {
+    float wv[VEC];
+    load_n<VEC>(w, wv);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] = v[i] * inv * wv[i];
+  };
+  auto emit_q = [&](int c, float (&v)[VEC]) {
+    scale(v, qinv, wq + c * VEC);
+    store_n<VEC>(cq + c * VEC, v);
+  };
+  auto emit_k = [&](int c, float (&v)[VEC]) {
+    scale(v, kinv, wkv + c * VEC);
+    if (pool_row) store_n<VEC>(pool_row + c * VEC, v);
+    if (c_out) store_n<VEC>(c_out + c * VEC, v);
+  };
+  if constexpr (NQ > 0) {
+#pragma unroll
+    for (int n = 0; n < NQ; ++n)
+      if (tid + n * kThreads < nq) emit_q(tid + n * kThreads, kq[n]);
+#pragma unroll
+    for (int n = 0; n < NK; ++n)
+      if (tid + n * kThreads < nk) emit_k(tid + n * kThreads, kk[n]);
+  } else {
+    for (int c = tid; c < nq; c += kThreads) { load_n<VEC>(zq + c * VEC, kq[0]); emit_q(c, kq[0]); }
+    for (int c = tid; c < nk; c += kThreads) { load_n<VEC>(zk + c * VEC, kk[0]); emit_k(c, kk[0]); }
   }
 }
 
@@ -339,7 +387,13 @@ cudaError_t launch_side_gate(const void* z, const void* side, const int64_t* tok
 template <typename T>
 cudaError_t launch_latent_prep(const LatentPrepArgs& a, cudaStream_t s) {
   if (a.rows == 0) return cudaSuccess;
-  latent_prep_kernel<T><<<(unsigned)a.rows, 128, 0, s>>>(a);
+  const unsigned g = (unsigned)a.rows;
+  const bool vec = a.q_rank % 8 == 0 && a.kv_rank % 8 == 0 && a.off_q % 8 == 0 && a.off_kv % 8 == 0 && a.down_stride % 8 == 0 &&
+                   a.pool_stride % 8 == 0 && aligned16(a.down) && aligned16(a.wq) && aligned16(a.wkv) && aligned16(a.cq) &&
+                   aligned16(a.c_out) && aligned16(a.pool);
+  if (vec && a.q_rank <= 8 * kThreads && a.kv_rank <= 8 * kThreads) latent_prep_kernel<T, 8, 1, 1><<<g, kThreads, 0, s>>>(a);
+  else if (vec) latent_prep_kernel<T, 8, 0, 0><<<g, kThreads, 0, s>>>(a);
+  else latent_prep_kernel<T, 1, 0, 0><<<g, kThreads, 0, s>>>(a);
   return cudaGetLastError();
 }
 
