@@ -100,9 +100,9 @@ class HybridLayer:
 
 @dataclass(frozen=True)
 class HybridConfig:
-    """A decoder whose layers each name their mixer and feed-forward.  Layers [loop_start, loop_stop) run `loop_times`
-    times in a row with the same weights; every pass has its own cache or state, and the embedding output is added to
-    the residual before each pass but the first."""
+    """A decoder whose layers each name their mixer and feed-forward.  The range [loop_start, loop_stop) is passed through
+    `loop_times` times with shared weights; passes share nothing they keep per request, and from the second one on the residual
+    first receives the token embeddings again."""
     vocab_size: int
     width: int
     layers: Tuple[HybridLayer, ...]
