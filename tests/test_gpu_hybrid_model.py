@@ -15,7 +15,7 @@ from oracle import berilix_oracle as orc
 
 pytestmark = pytest.mark.gpu
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
-TOL = {torch.float32: 3e-4, torch.bfloat16: 8e-2}        # root mean square over the vocabulary, relative to the spread
+TOL = {torch.float32: 3e-4, torch.bfloat16: 6e-2}        # root mean square over the vocabulary, relative to the spread
 CONFIGS = {"small": hc.small_config, "odd": hc.odd_config, "plain": hc.plain_config}
 
 
