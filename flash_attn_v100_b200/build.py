@@ -1,10 +1,12 @@
 """Build recipe for the sm_100a shared libraries (kept in-tree).
 
-`libfa_b200.so` (csrc/*.cu) holds the attention operators and the operators of the Qwen3-style decoder,
-`libfa_b200_hybrid.so` (csrc/hybrid/*.cu) those of the hybrid decoders, so that a process that serves one model
-builds and loads what that model needs.
+`libfa_b200.so` (csrc/*.cu) holds the attention operators and the operators of the Qwen3-style decoder; the hybrid
+decoders share `libfa_b200_rows.so` (csrc/rows/*.cu, row-wise operators) and have their mixers in
+`libfa_b200_hybrid.so` (csrc/hybrid/*.cu: decayed linear attention, latent attention) and `libfa_b200_mixers.so`
+(csrc/mixers/*.cu: gated recurrences, chunked attention).  A process that serves one model builds and loads what that
+model needs.
 
-    python -m flash_attn_v100_b200.build            # rebuild what is out of date, both libraries
+    python -m flash_attn_v100_b200.build            # rebuild what is out of date, all libraries
     python -m flash_attn_v100_b200.build --force
     python -m flash_attn_v100_b200.build -v         # also print ptxas resource usage
 
@@ -39,9 +41,9 @@ COMPILE_FLAGS = [
 LINK_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-shared", "-Xcompiler", "-fPIC"]
 
 
-HYBRID_CSRC = os.path.join(CSRC, "hybrid")
-HYBRID_LIB_PATH = os.path.join(PKG_DIR, "libfa_b200_hybrid.so")
-LIBRARIES = {"attention": (LIB_PATH, CSRC), "hybrid": (HYBRID_LIB_PATH, HYBRID_CSRC)}
+LIBRARIES = {"attention": (LIB_PATH, CSRC)}
+LIBRARIES.update({name: (os.path.join(PKG_DIR, f"libfa_b200_{name}.so"), os.path.join(CSRC, name))
+                  for name in ("rows", "hybrid", "mixers")})
 
 
 def sources(library: str = "attention"):
@@ -50,7 +52,7 @@ def sources(library: str = "attention"):
 
 
 def _headers():
-    deps = [os.path.join(d, f) for d in (CSRC, HYBRID_CSRC) for f in os.listdir(d) if f.endswith(".cuh")]
+    deps = [os.path.join(d, f) for _, d in LIBRARIES.values() for f in os.listdir(d) if f.endswith(".cuh")]
     deps += [os.path.join(INCLUDE, f) for f in os.listdir(INCLUDE)]
     return deps
 
@@ -104,7 +106,7 @@ def build(force: bool = False, verbose: bool = False, extra_flags=None, lib_path
         hdr_time = max(os.path.getmtime(h) for h in _headers())
         jobs, objs = [], []
         for src in sources(library):
-            obj = os.path.join(OBJ_DIR, f"{os.path.splitext(os.path.basename(src))[0]}.{tag}.o")
+            obj = os.path.join(OBJ_DIR, f"{library}.{os.path.splitext(os.path.basename(src))[0]}.{tag}.o")
             objs.append(obj)
             stale = force or verbose or not os.path.exists(obj) or \
                 os.path.getmtime(obj) < max(os.path.getmtime(src), hdr_time)

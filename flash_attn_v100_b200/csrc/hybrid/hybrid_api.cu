@@ -1,58 +1,16 @@
 // C-ABI entry points of the hybrid decoder's operators (see include/fa_b200_hybrid.h): argument checks and launches.
 #include "../../../include/fa_b200_hybrid.h"
 
-#include <cuda_runtime.h>
-#include <stdarg.h>
-#include <stdio.h>
-
+#include "../api_common.cuh"
 #include "hybrid_common.cuh"
 #include "latent_attention.cuh"
 #include "latent_prefill.cuh"
+#include "latent_prep.cuh"
 #include "lightning.cuh"
-#include "row_ops.cuh"
 
 namespace {
 
 using fa::hybrid::bf16;
-
-thread_local char g_err[512] = "";
-
-int fail(int code, const char* fmt, ...) {
-  va_list ap;
-  va_start(ap, fmt);
-  vsnprintf(g_err, sizeof(g_err), fmt, ap);
-  va_end(ap);
-  return code;
-}
-#define FAH_REQUIRE(cond, ...) \
-  do {                         \
-    if (!(cond)) return fail(FAH_ERR_INVALID_ARGUMENT, __VA_ARGS__); \
-  } while (0)
-
-int done(cudaError_t e, const char* what) {
-  if (e != cudaSuccess) return fail(FAH_ERR_CUDA, "%s failed: %s", what, cudaGetErrorString(e));
-  return FAH_OK;
-}
-bool dtype_ok(int dtype) { return dtype == FAH_F32 || dtype == FAH_BF16; }
-cudaStream_t st(void* s) { return static_cast<cudaStream_t>(s); }
-int sm_count() {
-  static int cached[64] = {0};
-  int dev = 0, n = 148;
-  if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return n;
-  if (cached[dev] == 0 && cudaDeviceGetAttribute(&n, cudaDevAttrMultiProcessorCount, dev) == cudaSuccess) cached[dev] = n;
-  return cached[dev] ? cached[dev] : n;
-}
-// cuTensorMapEncodeTiled, or null if the driver does not have it.
-void* tensor_map_encode() {
-  static void* fn = [] {
-    void* sym = nullptr;
-    cudaDriverEntryPointQueryResult qres;
-    const cudaError_t e = cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &sym, cudaEnableDefault, &qres);
-    return e == cudaSuccess && qres == cudaDriverEntryPointSuccess ? sym : nullptr;
-  }();
-  return fn;
-}
-constexpr int64_t kMaxRows = 1ll << 31;
 
 // Calls fn<T>(args...) for the element type of `dtype`.
 #define FAH_DISPATCH(dtype, fn, ...) ((dtype) == FAH_BF16 ? fn<bf16>(__VA_ARGS__) : fn<float>(__VA_ARGS__))
@@ -62,43 +20,6 @@ constexpr int64_t kMaxRows = 1ll << 31;
 extern "C" {
 
 const char* fah_last_error(void) { return g_err; }
-
-int fah_residual_norm(float* x, const void* delta, const void* delta_w, const void* embed, const int64_t* tokens, int embed_mode,
-                      int vocab, const void* w, void* out, int64_t rows, int cols, float eps, int dtype, void* stream) {
-  FAH_REQUIRE(dtype_ok(dtype), "unknown dtype %d", dtype);
-  FAH_REQUIRE(x != nullptr, "x is null");
-  FAH_REQUIRE(rows >= 0 && rows < kMaxRows && cols > 0, "bad sizes: rows=%lld cols=%d", (long long)rows, cols);
-  FAH_REQUIRE(embed_mode >= 0 && embed_mode <= 2, "embed_mode must be 0, 1 or 2");
-  FAH_REQUIRE(embed_mode == 0 || (embed != nullptr && tokens != nullptr && vocab > 0), "embed_mode %d needs embed, tokens and vocab", embed_mode);
-  FAH_REQUIRE(delta_w == nullptr || delta != nullptr, "delta_w without delta");
-  FAH_REQUIRE(w == nullptr || out != nullptr, "w without out");
-  fa::hybrid::ResidualNormArgs a{x, delta, delta_w, embed, tokens, embed_mode, w, out, rows, cols, vocab, eps};
-  return done(FAH_DISPATCH(dtype, fa::hybrid::launch_residual_norm, a, st(stream)), "residual_norm");
-}
-
-int fah_gated_norm(const void* o, const void* g, int64_t g_stride, const void* w, void* out, int64_t rows, int cols, float eps, int dtype,
-                   void* stream) {
-  FAH_REQUIRE(dtype_ok(dtype), "unknown dtype %d", dtype);
-  FAH_REQUIRE(o && g && w && out, "null pointer");
-  FAH_REQUIRE(rows >= 0 && rows < kMaxRows && cols > 0 && g_stride >= cols, "bad sizes: rows=%lld cols=%d", (long long)rows, cols);
-  return done(FAH_DISPATCH(dtype, fa::hybrid::launch_gated_norm, o, g, g_stride, w, out, rows, cols, eps, st(stream)), "gated_norm");
-}
-
-int fah_clamped_glu(const void* gu, void* out, int64_t rows, int n, float limit, float alpha, float shift, int dtype, void* stream) {
-  FAH_REQUIRE(dtype_ok(dtype), "unknown dtype %d", dtype);
-  FAH_REQUIRE(gu && out, "null pointer");
-  FAH_REQUIRE(rows >= 0 && rows < kMaxRows && n > 0, "bad sizes: rows=%lld n=%d", (long long)rows, n);
-  return done(FAH_DISPATCH(dtype, fa::hybrid::launch_clamped_glu, gu, out, rows, n, limit, alpha, shift, st(stream)), "clamped_glu");
-}
-
-int fah_side_gate(const void* z, const void* side, const int64_t* tokens, int vocab, int64_t side_stride, int off, void* out, int64_t rows,
-                  int n, int dtype, void* stream) {
-  FAH_REQUIRE(dtype_ok(dtype), "unknown dtype %d", dtype);
-  FAH_REQUIRE(z && side && tokens && out, "null pointer");
-  FAH_REQUIRE(rows >= 0 && rows < kMaxRows && n > 0 && vocab > 0 && off >= 0 && off + (int64_t)n <= side_stride, "bad sizes: rows=%lld n=%d off=%d",
-              (long long)rows, n, off);
-  return done(FAH_DISPATCH(dtype, fa::hybrid::launch_side_gate, z, side, tokens, vocab, side_stride, off, out, rows, n, st(stream)), "side_gate");
-}
 
 size_t fah_lightning_workspace(int n_seq, int heads, int dk, int dv, int max_len, int dtype) {
   if (dtype != FAH_BF16 || n_seq <= 0 || heads <= 0 || dk <= 0 || dv <= 0 || max_len <= 0) return 0;
@@ -110,13 +31,13 @@ size_t fah_lightning_workspace(int n_seq, int heads, int dk, int dv, int max_len
 int fah_lightning(const void* qkv, int64_t stride, int off_q, int off_k, int off_v, int heads, int dk, int dv, const float* decay, float* state,
                   int n_slots, const int32_t* slots, const int32_t* starts, const int32_t* cu_seqlens, int n_seq, int max_len, int64_t tokens,
                   void* out, void* workspace, size_t workspace_bytes, int32_t* status, int dtype, void* stream) {
-  FAH_REQUIRE(dtype_ok(dtype), "unknown dtype %d", dtype);
-  FAH_REQUIRE(qkv && decay && state && slots && starts && out && status, "null pointer");
-  FAH_REQUIRE(heads > 0 && heads < 65536 && dk > 0 && dv > 0 && n_slots > 0, "bad sizes: heads=%d dk=%d dv=%d slots=%d", heads, dk, dv, n_slots);
-  FAH_REQUIRE(dk <= 1536, "dk=%d is larger than the 1536 the kernels are built for", dk);
-  FAH_REQUIRE(n_seq >= 0 && tokens >= n_seq && tokens < kMaxRows && (cu_seqlens != nullptr || tokens == n_seq), "bad sizes: n_seq=%d tokens=%lld", n_seq,
+  FA_REQUIRE(dtype_ok(dtype), "unknown dtype %d", dtype);
+  FA_REQUIRE(qkv && decay && state && slots && starts && out && status, "null pointer");
+  FA_REQUIRE(heads > 0 && heads < 65536 && dk > 0 && dv > 0 && n_slots > 0, "bad sizes: heads=%d dk=%d dv=%d slots=%d", heads, dk, dv, n_slots);
+  FA_REQUIRE(dk <= 1536, "dk=%d is larger than the 1536 the kernels are built for", dk);
+  FA_REQUIRE(n_seq >= 0 && tokens >= n_seq && tokens < kMaxRows && (cu_seqlens != nullptr || tokens == n_seq), "bad sizes: n_seq=%d tokens=%lld", n_seq,
               (long long)tokens);
-  FAH_REQUIRE(off_q >= 0 && off_k >= 0 && off_v >= 0 && off_q + (int64_t)heads * dk <= stride && off_k + (int64_t)heads * dk <= stride &&
+  FA_REQUIRE(off_q >= 0 && off_k >= 0 && off_v >= 0 && off_q + (int64_t)heads * dk <= stride && off_k + (int64_t)heads * dk <= stride &&
                   off_v + (int64_t)heads * dv <= stride,
               "a column range ends past the row stride");
   fa::hybrid::LightningArgs a{};
@@ -126,9 +47,9 @@ int fah_lightning(const void* qkv, int64_t stride, int off_q, int off_k, int off
   if (fa::hybrid::lightning_decode_supported(a))
     return done(FAH_DISPATCH(dtype, fa::hybrid::launch_lightning_decode, a, sm_count(), st(stream)), "lightning_decode");
   if (dtype == FAH_BF16 && fa::hybrid::lightning_chunk_supported(a)) {
-    FAH_REQUIRE(max_len > 0, "prompts need max_len");
+    FA_REQUIRE(max_len > 0, "prompts need max_len");
     const size_t need = fah_lightning_workspace(n_seq, heads, dk, dv, max_len, dtype);
-    FAH_REQUIRE(workspace_bytes >= need && (need == 0 || (workspace != nullptr && (reinterpret_cast<uintptr_t>(workspace) & 15) == 0)),
+    FA_REQUIRE(workspace_bytes >= need && (need == 0 || (workspace != nullptr && (reinterpret_cast<uintptr_t>(workspace) & 15) == 0)),
                 "the workspace has %zu bytes, %zu (16-byte aligned) are needed", workspace_bytes, need);
     a.max_segs = fa::hybrid::lightning_segments(n_seq, heads, dk, dv, max_len, sm_count(), &a.seg_len);
     a.seg_state = static_cast<float*>(workspace);
@@ -141,13 +62,13 @@ int fah_latent_prep(const void* down, int64_t down_stride, int off_q, int q_rank
                     const void* wkv, float eps, const float* cos_t, const float* sin_t, void* cq, void* c_out, void* r_out, void* pool,
                     int pool_stride, int n_blocks, const int32_t* block_table, int max_blocks, int n_seq, const int32_t* tok_seq,
                     const int32_t* positions, int64_t rows, int32_t* status, int dtype, void* stream) {
-  FAH_REQUIRE(dtype_ok(dtype), "unknown dtype %d", dtype);
-  FAH_REQUIRE(down && wq && wkv && cos_t && sin_t && cq && pool && block_table && tok_seq && positions && status, "null pointer");
-  FAH_REQUIRE(q_rank > 0 && kv_rank > 0 && rot_dim > 0 && rot_dim % 2 == 0, "bad sizes: q_rank=%d kv_rank=%d rot_dim=%d", q_rank, kv_rank, rot_dim);
-  FAH_REQUIRE(off_q >= 0 && off_kv >= 0 && off_r >= 0 && off_q + (int64_t)q_rank <= down_stride && off_kv + (int64_t)kv_rank <= down_stride &&
+  FA_REQUIRE(dtype_ok(dtype), "unknown dtype %d", dtype);
+  FA_REQUIRE(down && wq && wkv && cos_t && sin_t && cq && pool && block_table && tok_seq && positions && status, "null pointer");
+  FA_REQUIRE(q_rank > 0 && kv_rank > 0 && rot_dim > 0 && rot_dim % 2 == 0, "bad sizes: q_rank=%d kv_rank=%d rot_dim=%d", q_rank, kv_rank, rot_dim);
+  FA_REQUIRE(off_q >= 0 && off_kv >= 0 && off_r >= 0 && off_q + (int64_t)q_rank <= down_stride && off_kv + (int64_t)kv_rank <= down_stride &&
                   off_r + (int64_t)rot_dim <= down_stride,
               "a column range ends past the row stride");
-  FAH_REQUIRE(pool_stride >= kv_rank + rot_dim && n_blocks > 0 && max_blocks > 0 && n_seq > 0 && rows >= 0 && rows < kMaxRows, "bad cache sizes");
+  FA_REQUIRE(pool_stride >= kv_rank + rot_dim && n_blocks > 0 && max_blocks > 0 && n_seq > 0 && rows >= 0 && rows < kMaxRows, "bad cache sizes");
   fa::hybrid::LatentPrepArgs a{down, down_stride, off_q, q_rank, off_kv, kv_rank, off_r, rot_dim, wq, wkv, eps, cos_t, sin_t, cq, c_out, r_out, pool,
                                pool_stride, n_blocks, block_table, max_blocks, n_seq, tok_seq, positions, rows, status};
   return done(FAH_DISPATCH(dtype, fa::hybrid::launch_latent_prep, a, st(stream)), "latent_prep");
@@ -155,9 +76,9 @@ int fah_latent_prep(const void* down, int64_t down_stride, int off_q, int q_rank
 
 int fah_rotate_heads(void* q, const float* cos_t, const float* sin_t, int64_t rows, int heads, int head_stride, int off, int rot_dim, int dtype,
                      void* stream) {
-  FAH_REQUIRE(dtype_ok(dtype), "unknown dtype %d", dtype);
-  FAH_REQUIRE(q && cos_t && sin_t, "null pointer");
-  FAH_REQUIRE(rows >= 0 && rows < kMaxRows && heads > 0 && off >= 0 && rot_dim >= 0 && rot_dim % 2 == 0 && off + rot_dim <= head_stride,
+  FA_REQUIRE(dtype_ok(dtype), "unknown dtype %d", dtype);
+  FA_REQUIRE(q && cos_t && sin_t, "null pointer");
+  FA_REQUIRE(rows >= 0 && rows < kMaxRows && heads > 0 && off >= 0 && rot_dim >= 0 && rot_dim % 2 == 0 && off + rot_dim <= head_stride,
               "bad sizes: heads=%d off=%d rot_dim=%d head_stride=%d", heads, off, rot_dim, head_stride);
   return done(FAH_DISPATCH(dtype, fa::hybrid::launch_rotate_heads, q, cos_t, sin_t, rows, heads, head_stride, off, rot_dim, st(stream)), "rotate_heads");
 }
@@ -172,12 +93,12 @@ int fah_latent_attention(const void* q_abs, const void* q, int q_stride, int q_o
                          int pool_stride, int n_blocks, const int32_t* block_table, int max_blocks, int n_seq, const int32_t* tok_seq,
                          const int32_t* positions, const void* gate, int64_t gate_stride, int heads, int kv_rank, int rot_dim, float scale, void* out,
                          int64_t rows, void* workspace, size_t workspace_bytes, int32_t* status, int dtype, void* stream) {
-  FAH_REQUIRE(dtype_ok(dtype), "unknown dtype %d", dtype);
-  FAH_REQUIRE(q_abs && q && cos_t && sin_t && pool && block_table && tok_seq && positions && out && status, "null pointer");
-  FAH_REQUIRE(heads > 0 && heads < 65536 && kv_rank > 0 && kv_rank <= 16384 && rot_dim >= 0 && rot_dim % 2 == 0 && q_off >= 0 && q_off + rot_dim <= q_stride,
+  FA_REQUIRE(dtype_ok(dtype), "unknown dtype %d", dtype);
+  FA_REQUIRE(q_abs && q && cos_t && sin_t && pool && block_table && tok_seq && positions && out && status, "null pointer");
+  FA_REQUIRE(heads > 0 && heads < 65536 && kv_rank > 0 && kv_rank <= 16384 && rot_dim >= 0 && rot_dim % 2 == 0 && q_off >= 0 && q_off + rot_dim <= q_stride,
               "bad sizes: heads=%d kv_rank=%d rot_dim=%d", heads, kv_rank, rot_dim);
-  FAH_REQUIRE(pool_stride >= kv_rank + rot_dim && n_blocks > 0 && max_blocks > 0 && n_seq > 0 && rows >= 0 && rows < kMaxRows, "bad cache sizes");
-  FAH_REQUIRE(gate == nullptr || gate_stride >= heads, "gate_stride=%lld is smaller than heads=%d", (long long)gate_stride, heads);
+  FA_REQUIRE(pool_stride >= kv_rank + rot_dim && n_blocks > 0 && max_blocks > 0 && n_seq > 0 && rows >= 0 && rows < kMaxRows, "bad cache sizes");
+  FA_REQUIRE(gate == nullptr || gate_stride >= heads, "gate_stride=%lld is smaller than heads=%d", (long long)gate_stride, heads);
   fa::hybrid::LatentAttentionArgs a{};
   a.q_abs = q_abs; a.q = q; a.q_stride = q_stride; a.q_off = q_off; a.cos_t = cos_t; a.sin_t = sin_t; a.pool = pool; a.pool_stride = pool_stride;
   a.n_blocks = n_blocks; a.block_table = block_table; a.max_blocks = max_blocks; a.n_seq = n_seq; a.tok_seq = tok_seq; a.positions = positions;
@@ -185,7 +106,7 @@ int fah_latent_attention(const void* q_abs, const void* q, int q_stride, int q_o
   a.status = status;
   if (dtype == FAH_BF16 && fa::hybrid::latent_decode_supported(a)) {
     const size_t need = fah_latent_attention_workspace(heads, kv_rank, rot_dim, rows, dtype);
-    FAH_REQUIRE(workspace_bytes >= need && (need == 0 || (workspace != nullptr && (reinterpret_cast<uintptr_t>(workspace) & 15) == 0)),
+    FA_REQUIRE(workspace_bytes >= need && (need == 0 || (workspace != nullptr && (reinterpret_cast<uintptr_t>(workspace) & 15) == 0)),
                 "the workspace has %zu bytes, %zu (16-byte aligned) are needed", workspace_bytes, need);
     a.n_cta = fa::hybrid::latent_decode_ctas(heads, sm_count());
     a.part_o = static_cast<float*>(workspace);
@@ -205,14 +126,14 @@ int fah_latent_prefill_supported(int dim, int rot_dim, int vdim, float scale, in
 int fah_latent_prefill(const void* q, const void* kv, const void* kr, const void* gate, int64_t gate_stride, const int32_t* cu_q,
                        const int32_t* cu_kv, int n_seq, int max_q, int64_t total_q, int64_t total_kv, int heads, int dim, int rot_dim, int vdim,
                        float scale, void* out, int32_t* status, void* stream) {
-  FAH_REQUIRE(q && kv && kr && cu_q && cu_kv && out && status, "null pointer");
+  FA_REQUIRE(q && kv && kr && cu_q && cu_kv && out && status, "null pointer");
   if (!fa::hybrid::latent_prefill_supported(dim, rot_dim, vdim, scale))
     return fail(FAH_ERR_UNSUPPORTED, "latent_prefill is not built for dim=%d rot_dim=%d vdim=%d scale=%g", dim, rot_dim, vdim, (double)scale);
-  FAH_REQUIRE(heads > 0 && n_seq > 0 && max_q > 0 && total_q >= 0 && total_q < kMaxRows && total_kv >= total_q && total_kv < kMaxRows,
+  FA_REQUIRE(heads > 0 && n_seq > 0 && max_q > 0 && total_q >= 0 && total_q < kMaxRows && total_kv >= total_q && total_kv < kMaxRows,
               "bad sizes: heads=%d n_seq=%d max_q=%d total_q=%lld total_kv=%lld", heads, n_seq, max_q, (long long)total_q, (long long)total_kv);
-  FAH_REQUIRE(gate == nullptr || gate_stride >= heads, "gate_stride=%lld is smaller than heads=%d", (long long)gate_stride, heads);
+  FA_REQUIRE(gate == nullptr || gate_stride >= heads, "gate_stride=%lld is smaller than heads=%d", (long long)gate_stride, heads);
   for (const void* p : {q, kv, kr, (const void*)out})
-    FAH_REQUIRE((reinterpret_cast<uintptr_t>(p) & 15) == 0, "q, kv, kr and out must be 16-byte aligned");
+    FA_REQUIRE((reinterpret_cast<uintptr_t>(p) & 15) == 0, "q, kv, kr and out must be 16-byte aligned");
   void* enc = tensor_map_encode();
   if (enc == nullptr) return fail(FAH_ERR_CUDA, "cuTensorMapEncodeTiled is not available from the driver");
   fa::hybrid::LatentPrefillArgs a{q, kv, kr, gate, gate_stride, cu_q, cu_kv, n_seq, max_q, total_q, total_kv, heads, dim, rot_dim, vdim, scale, out,
@@ -222,9 +143,9 @@ int fah_latent_prefill(const void* q, const void* kv, const void* kr, const void
 
 int fah_latent_gather(const void* pool, int pool_stride, int n_blocks, const int32_t* block_table, int max_blocks, int n_seq, const int32_t* cu_kv,
                       int64_t total_kv, int kv_rank, int rot_dim, void* c, void* r, int32_t* status, int dtype, void* stream) {
-  FAH_REQUIRE(dtype_ok(dtype), "unknown dtype %d", dtype);
-  FAH_REQUIRE(pool && block_table && cu_kv && c && r && status, "null pointer");
-  FAH_REQUIRE(kv_rank > 0 && rot_dim > 0 && pool_stride >= kv_rank + rot_dim && n_blocks > 0 && max_blocks > 0 && n_seq > 0 && total_kv >= 0 &&
+  FA_REQUIRE(dtype_ok(dtype), "unknown dtype %d", dtype);
+  FA_REQUIRE(pool && block_table && cu_kv && c && r && status, "null pointer");
+  FA_REQUIRE(kv_rank > 0 && rot_dim > 0 && pool_stride >= kv_rank + rot_dim && n_blocks > 0 && max_blocks > 0 && n_seq > 0 && total_kv >= 0 &&
                   total_kv < kMaxRows,
               "bad sizes: kv_rank=%d rot_dim=%d n_seq=%d total_kv=%lld", kv_rank, rot_dim, n_seq, (long long)total_kv);
   fa::hybrid::LatentGatherArgs a{pool, pool_stride, n_blocks, block_table, max_blocks, n_seq, cu_kv, total_kv, kv_rank, rot_dim, c, r, status};

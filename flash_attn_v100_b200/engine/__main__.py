@@ -20,12 +20,11 @@ def main(argv=None) -> int:
     ap.add_argument("--prefill-portion", type=int, default=0, help="most tokens of a prompt per pass (0: the whole prompt)")
     args = ap.parse_args(argv)
     import torch
-    from ..build import build
     from . import registry
     from .runner import GenerationRunner
     prompts = [[int(t) for t in p.split(",")] for p in args.prompt]
     raw = registry.read_config(args.model)
-    build(library=registry.family_of(raw).library)
+    registry.family_of(raw).build_libraries()
     model = registry.load_model(args.model, getattr(torch, args.dtype) if args.dtype else None, config=raw)
     groups = {}
     for i, p in enumerate(prompts):

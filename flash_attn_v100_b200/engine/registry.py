@@ -9,16 +9,22 @@ from typing import Callable, Dict, Tuple
 import torch
 
 from . import safetensors
-from .config import HybridConfig, ModelConfig
+from .config import HybridConfig, ModelConfig, sabipel_config
 
 
 @dataclass(frozen=True)
 class ModelFamily:
     architecture: str
-    library: str                                  # the CUDA library of its operators (see build.LIBRARIES)
+    libraries: Tuple[str, ...]                    # the CUDA libraries of its operators (see build.LIBRARIES)
     dtypes: Tuple[torch.dtype, ...]               # activation types it runs in, the default first
     config_from_dict: Callable
     build: Callable                               # (cfg, tensors, dtype, device) -> model
+
+    def build_libraries(self) -> None:
+        """Compile what is out of date of the libraries this family needs, and of no other."""
+        from ..build import build
+        for name in self.libraries:
+            build(library=name)
 
 
 _FAMILIES: Dict[str, ModelFamily] = {}
@@ -70,5 +76,6 @@ def _build_hybrid(cfg, tensors, dtype, device):
     return HybridDecoder(cfg, hybrid_weights(cfg, tensors, dtype, device), device=device)
 
 
-register(ModelFamily("Qwen3", "attention", (torch.bfloat16,), ModelConfig.from_dict, _build_qwen3))
-register(ModelFamily("Berilix", "hybrid", (torch.bfloat16, torch.float32), HybridConfig.from_dict, _build_hybrid))
+register(ModelFamily("Qwen3", ("attention",), (torch.bfloat16,), ModelConfig.from_dict, _build_qwen3))
+register(ModelFamily("Berilix", ("rows", "hybrid"), (torch.bfloat16, torch.float32), HybridConfig.from_dict, _build_hybrid))
+register(ModelFamily("Sabipel", ("rows", "mixers"), (torch.bfloat16, torch.float32), sabipel_config, _build_hybrid))

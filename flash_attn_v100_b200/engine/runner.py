@@ -15,8 +15,11 @@ class GenerationRunner:
     def __init__(self, model, max_batch: int, max_seq_len: int, use_cuda_graph: bool = True,
                  peer_collectives: bool = False, num_blocks: int = 0):
         """`model`: a TPDecoder or HybridDecoder.  `num_blocks`: cache blocks shared by the requests (default: enough
-        for `max_batch` requests of `max_seq_len` tokens)."""
+        for `max_batch` requests of `max_seq_len` tokens).  A model with a table of positions bounds `max_seq_len`."""
         cfg = model.cfg
+        limit = getattr(model, "max_positions", 0)
+        if limit:
+            max_seq_len = min(max_seq_len, limit)
         self.model = model
         self.max_batch, self.max_seq_len = max_batch, max_seq_len
         self.max_blocks = (max_seq_len + 15) // 16
@@ -129,7 +132,8 @@ class GenerationRunner:
         `logits_out` (a list, eager mode only) receives this rank's logits of every step."""
         m, kv, dev = self.model, self.kv, self.model.device
         B, P = prompts.shape
-        assert B <= self.max_batch and P + max_new_tokens <= self.max_seq_len
+        if B > self.max_batch or P + max_new_tokens > self.max_seq_len:
+            raise ValueError(f"{B} requests of {P} + {max_new_tokens} tokens do not fit max_batch={self.max_batch}, max_seq_len={self.max_seq_len}")
         if prefill_portion and not m.supports_portions:
             raise ValueError(f"{type(m).__name__} takes a prompt in one pass")
         ids = [f"r{i}" for i in range(B)]

@@ -27,7 +27,6 @@ def main(argv=None) -> int:
     ap.add_argument("--max-tokens", type=int, required=True, help="most tokens that live requests hold at any time")
     args = ap.parse_args(argv)
     import torch
-    from ..build import build
     from ..kv_cache import BLOCK_SIZE
     from . import registry
     from .runner import GenerationRunner
@@ -37,7 +36,7 @@ def main(argv=None) -> int:
     if dtype not in family.dtypes:
         print(f"{family.architecture} does not run in {args.dtype}", file=sys.stderr)
         return EXIT_NO_SUCH_TYPE
-    build(library=family.library)
+    family.build_libraries()
     model = registry.load_model(args.model, dtype, config=raw)
     blocks = (args.max_tokens + BLOCK_SIZE - 1) // BLOCK_SIZE + MAX_REQUESTS      # every request may leave a block part filled
     runner = GenerationRunner(model, max_batch=MAX_REQUESTS, max_seq_len=max(args.max_tokens, 1), num_blocks=blocks)

@@ -14,7 +14,8 @@ from typing import Dict, List
 
 import torch
 
-from .config import HybridConfig, LightningSpec, ModelConfig
+from .config import (ChunkedAttentionSpec, ClampedGluSpec, HybridConfig, LatentAttentionSpec, LightningSpec, Mamba2Spec, MlstmSpec,
+                     ModelConfig)
 
 
 def _randn(shape, gen, std, device, dtype):
@@ -101,41 +102,71 @@ def rank_weights_from_tensors(cfg: ModelConfig, tensors: Dict[str, torch.Tensor]
 
 
 # ---- hybrid decoders -------------------------------------------------------------------------------------------
+def _mixer_shapes(m, W: int) -> Dict[str, tuple]:
+    if isinstance(m, LightningSpec):
+        kd, vd = m.heads * m.dim, m.heads * m.vdim
+        return {"q": (kd, W), "k": (kd, W), "v": (vd, W), "g": (vd, W), "o": (W, vd), "norm": (vd,)}
+    if isinstance(m, LatentAttentionSpec):
+        H = m.heads
+        return {"dq": (m.q_rank, W), "dq.norm": (m.q_rank,), "uq": (H * (m.dim + m.rot_dim), m.q_rank),
+                "dkv": (m.kv_rank + m.rot_dim, W), "dkv.norm": (m.kv_rank,), "uk": (H * m.dim, m.kv_rank),
+                "uv": (H * m.vdim, m.kv_rank), "g": (H, W), "o": (W, H * m.vdim)}
+    if isinstance(m, MlstmSpec):
+        kd, vd, H = m.heads * m.dim, m.heads * m.vdim, (m.heads,)
+        return {"q": (kd, W), "k": (kd, W), "v": (vd, W), "g": (vd, W), "o": (W, vd), "norm": (vd,),
+                "i": H + (W,), "i.b": H, "f": H + (W,), "f.b": H}
+    if isinstance(m, Mamba2Spec):
+        H = (m.heads,)
+        return {"in": (m.inner + m.channels + m.heads, W), "conv": (m.channels, m.conv), "conv.b": (m.channels,), "dt_bias": H, "A_log": H,
+                "D": H, "norm": (m.inner,), "o": (W, m.inner)}
+    if isinstance(m, ChunkedAttentionSpec):
+        qd, kd, vd = m.heads * m.dim, m.kv_heads * m.dim, m.heads * m.vdim
+        out = {"q": (qd, W), "k": (kd, W), "v": (m.kv_heads * m.vdim, W), "q.norm": (qd,), "k.norm": (kd,), "g": (vd, W), "o": (W, vd)}
+        return dict(out, vmix=()) if m.v_mix else out
+    raise TypeError(type(m))
+
+
 def hybrid_tensor_shapes(cfg: HybridConfig) -> Dict[str, tuple]:
     """Name and shape of every tensor of the model."""
     W = cfg.width
     out = {"embed": (cfg.vocab_size, W), "final.norm": (W,)}
+    if cfg.bigram is not None:
+        out["bigram"] = (cfg.bigram.buckets + 1, W)
+    if cfg.max_positions:
+        out["pos"] = (cfg.max_positions, W)
     if cfg.side_dim:
         out["side.embed"] = (cfg.vocab_size, len(cfg.layers) * cfg.side_dim)
     for i, layer in enumerate(cfg.layers):
-        m, pre = layer.mixer, f"l{i}."
+        pre = f"l{i}."
         out[pre + "norm1"] = (W,)
-        if isinstance(m, LightningSpec):
-            kd, vd = m.heads * m.dim, m.heads * m.vdim
-            mix = {"q": (kd, W), "k": (kd, W), "v": (vd, W), "g": (vd, W), "o": (W, vd), "norm": (vd,)}
-        else:
-            H = m.heads
-            mix = {"dq": (m.q_rank, W), "dq.norm": (m.q_rank,), "uq": (H * (m.dim + m.rot_dim), m.q_rank),
-                   "dkv": (m.kv_rank + m.rot_dim, W), "dkv.norm": (m.kv_rank,), "uk": (H * m.dim, m.kv_rank),
-                   "uv": (H * m.vdim, m.kv_rank), "g": (H, W), "o": (W, H * m.vdim)}
-        out.update({pre + "mix." + k: s for k, s in mix.items()})
+        out.update({pre + "mix." + k: s for k, s in _mixer_shapes(layer.mixer, W).items()})
         if layer.mlp is not None:
             F = layer.mlp.ff
-            out.update({pre + "norm2": (W,), pre + "mlp.gate": (F, W), pre + "mlp.up": (F, W), pre + "mlp.down": (W, F)})
+            gate = {pre + "mlp.gate": (F, W)} if isinstance(layer.mlp, ClampedGluSpec) else {}
+            out.update({pre + "norm2": (W,), **gate, pre + "mlp.up": (F, W), pre + "mlp.down": (W, F)})
         if cfg.side_dim:
             out.update({pre + "side.gate": (cfg.side_dim, W), pre + "side.proj": (W, cfg.side_dim), pre + "side.norm": (W,)})
     return out
 
 
 def random_hybrid_tensors(cfg: HybridConfig, seed: int, device="cpu", dtype=torch.bfloat16) -> Dict[str, torch.Tensor]:
-    """Seeded random tensors: matrices N(0, 1 / inputs), norm weights 1 + N(0, 0.1^2), embeddings N(0, 1)."""
+    """Seeded random tensors: matrices N(0, 1 / inputs), norm weights 1 + N(0, 0.1^2), embeddings N(0, 1); gate biases 3 + N(0, 0.1^2)
+    (forget) and N(0, 0.1^2), step biases around softplus^-1(0.05), decay rates 1 to 16, mixing weights 1 / 2."""
     g = torch.Generator(device=device).manual_seed(seed)
     out = {}
     for name, shape in hybrid_tensor_shapes(cfg).items():
         t = torch.randn(shape, generator=g, device=device)
-        if len(shape) == 1:
+        if len(shape) == 0:
+            t = torch.tensor(0.5)
+        elif name.endswith((".f.b", ".i.b", ".conv.b")):
+            t = 0.1 * t + (3.0 if name.endswith(".f.b") else 0.0)
+        elif name.endswith(".dt_bias"):
+            t = 0.1 * t - 3.0
+        elif name.endswith(".A_log"):
+            t = torch.rand(shape, generator=g, device=device) * 2.77
+        elif len(shape) == 1:
             t = 1.0 + 0.1 * t
-        elif not name.endswith("embed"):
+        elif name not in ("embed", "side.embed", "bigram", "pos"):
             t = t / shape[1] ** 0.5
         out[name] = t.to(dtype)
     return out
@@ -157,9 +188,11 @@ def _stack(mats, multiple: int = 8):
 
 def hybrid_weights(cfg: HybridConfig, tensors: Dict[str, torch.Tensor], dtype, device):
     """The model's tensors in the layout the decoder runs: projections of the same input stacked into one matrix.
-    {'embed', 'side_embed', 'final_norm', 'layers': [dict per layer]}."""
+    {'embed', 'side_embed', 'bigram', 'pos', 'final_norm', 'layers': [dict per layer]}.  In parallel layers the output projections of
+    mixer and feed-forward are one matrix over their activations side by side."""
     want = hybrid_tensor_shapes(cfg)
-    missing, extra = sorted(set(want) - set(tensors)), sorted(set(tensors) - set(want))
+    unused = {f"l{i}.mix.vmix" for i in range(len(cfg.layers))}           # of a layer that does not mix values
+    missing, extra = sorted(set(want) - set(tensors)), sorted(set(tensors) - set(want) - unused)
     if missing or extra:
         raise ValueError(f"tensors do not fit the configuration: missing {missing[:5]}, unknown {extra[:5]}")
     for name, shape in want.items():
@@ -173,11 +206,25 @@ def hybrid_weights(cfg: HybridConfig, tensors: Dict[str, torch.Tensor], dtype, d
     for i, layer in enumerate(cfg.layers):
         m, pre = layer.mixer, f"l{i}."
         mix = lambda n: get(pre + "mix." + n)
+        f32 = lambda n: tensors[pre + "mix." + n].to(device=device, dtype=torch.float32).contiguous()
         lw = {"norm1": get(pre + "norm1")}
         if isinstance(m, LightningSpec):
             lw["w_in"], lw["in_at"] = _stack([mix(n) for n in ("q", "k", "v", "g")])
             lw["norm"], lw["w_out"] = mix("norm"), mix("o")
             lw["decay"] = torch.tensor(m.decay, dtype=torch.float32, device=device)
+        elif isinstance(m, MlstmSpec):
+            lw["w_in"], lw["in_at"] = _stack([mix(n) for n in ("q", "k", "v", "g", "i", "f")])
+            lw["norm"], lw["w_out"], lw["bias_i"], lw["bias_f"] = mix("norm"), mix("o"), mix("i.b"), mix("f.b")
+        elif isinstance(m, Mamba2Spec):
+            lw["w_in"], _ = _stack([mix("in")])
+            lw["conv_w"], lw["conv_b"] = mix("conv").t().contiguous(), mix("conv.b")
+            lw["dt_bias"], lw["a_log"], lw["skip"] = f32("dt_bias"), f32("A_log"), f32("D")
+            lw["norm"], lw["w_out"] = mix("norm"), mix("o")
+        elif isinstance(m, ChunkedAttentionSpec):
+            lw["w_in"], lw["in_at"] = _stack([mix(n) for n in ("q", "k", "v", "g")])
+            lw["q_norm"], lw["k_norm"], lw["w_out"] = mix("q.norm"), mix("k.norm"), mix("o")
+            lw["lambda"] = float(tensors[pre + "mix.vmix"].float()) if m.v_mix else 0.0
+            lw["slopes"] = torch.tensor(m.slopes, dtype=torch.float32, device=device)
         else:
             dkv = mix("dkv")
             lw["w_in"], lw["in_at"] = _stack([mix("dq"), dkv[:m.kv_rank], dkv[m.kv_rank:], mix("g")])
@@ -188,10 +235,17 @@ def hybrid_weights(cfg: HybridConfig, tensors: Dict[str, torch.Tensor], dtype, d
             lw["w_uv"] = lw["w_ukv"][m.heads * m.dim:].view(m.heads, m.vdim, m.kv_rank)
         if layer.mlp is not None:
             lw["norm2"] = get(pre + "norm2")
-            lw["w_gu"] = torch.cat([get(pre + "mlp.gate"), get(pre + "mlp.up")]).contiguous()
-            lw["w_down"] = get(pre + "mlp.down")
+            if isinstance(layer.mlp, ClampedGluSpec):
+                lw["w_gu"] = torch.cat([get(pre + "mlp.gate"), get(pre + "mlp.up")]).contiguous()
+            else:
+                lw["w_up"] = get(pre + "mlp.up")
+            if cfg.parallel:
+                lw["w_out"] = torch.cat([lw["w_out"], get(pre + "mlp.down")], dim=1).contiguous()
+            else:
+                lw["w_down"] = get(pre + "mlp.down")
         if cfg.side_dim:
             lw["side_gate"], lw["side_proj"], lw["side_norm"] = (get(pre + "side." + n) for n in ("gate", "proj", "norm"))
         layers.append(lw)
     return {"embed": get("embed"), "side_embed": get("side.embed") if cfg.side_dim else None,
+            "bigram": get("bigram") if cfg.bigram is not None else None, "pos": get("pos") if cfg.max_positions else None,
             "final_norm": get("final.norm"), "layers": layers}

@@ -2,108 +2,15 @@
 stream.  T is the activation type, bfloat16 or float32; there is no CPU path."""
 from __future__ import annotations
 
-import ctypes
-
 import torch
 
 from . import _lib
-
-_DTYPE = {torch.float32: 0, torch.bfloat16: 1}
-
-
-def _p(t):
-    return None if t is None else ctypes.c_void_p(t.data_ptr())
+from .row_ops import _DTYPE, _check, _p, _stream, _type, _workspace
+from .row_ops import clamped_glu, gated_norm, residual_norm, side_gate  # noqa: F401  (the row-wise operators of the same decoder)
 
 
-def _stream(t):
-    return ctypes.c_void_p(torch.cuda.current_stream(t.device).cuda_stream)
-
-
-def _check(t, name, dtype, contiguous=True):
-    if not t.is_cuda:
-        raise RuntimeError(f"{name} must be a CUDA tensor")
-    if t.dtype != dtype:
-        raise RuntimeError(f"{name} must be {dtype}, got {t.dtype}")
-    if contiguous and not t.is_contiguous():
-        raise RuntimeError(f"{name} must be contiguous")
-
-
-def _workspace(nbytes, device):
-    return torch.empty(nbytes, dtype=torch.uint8, device=device) if nbytes else None
-
-
-def _type(t, name):
-    if t.dtype not in _DTYPE:
-        raise RuntimeError(f"{name} must be bfloat16 or float32, got {t.dtype}")
-    return t.dtype
-
-
-def residual_norm(x, w=None, eps=1e-5, *, delta=None, delta_w=None, embed=None, tokens=None, init=False, out=True, dtype=None):
-    """x [rows, cols] fp32, in place: x = embed[tokens] (`init`) or x += embed[tokens], then x += delta or
-    x += rmsnorm(delta) * delta_w.  Returns rmsnorm(x) * w, or x itself when w is None, in the activation type; None when
-    `out` is False."""
-    _check(x, "x", torch.float32)
-    like = next((t for t in (delta, embed, w) if t is not None), None)
-    T = dtype or (_type(like, "delta / embed / w") if like is not None else None)
-    if T is None:
-        raise RuntimeError("residual_norm needs dtype when neither delta, embed nor w is given")
-    for name, t in (("delta", delta), ("delta_w", delta_w), ("embed", embed), ("w", w)):
-        if t is not None:
-            _check(t, name, T)
-    rows, cols = x.shape
-    if delta is not None and delta.shape != x.shape:
-        raise RuntimeError("delta must have the shape of x")
-    for name, t in (("delta_w", delta_w), ("w", w)):
-        if t is not None and t.numel() != cols:
-            raise RuntimeError(f"{name} must have {cols} elements")
-    if embed is not None:
-        _check(tokens, "tokens", torch.int64)
-        if tokens.numel() != rows or embed.size(1) != cols:
-            raise RuntimeError("tokens must have one entry per row and embed the width of x")
-    res = torch.empty((rows, cols), dtype=T, device=x.device) if out else None
-    mode = 0 if embed is None else (2 if init else 1)
-    _lib.check_hybrid(_lib.load_hybrid().fah_residual_norm(
-        _p(x), _p(delta), _p(delta_w), _p(embed), _p(tokens) if embed is not None else None, mode,
-        embed.size(0) if embed is not None else 0, _p(w) if out else None, _p(res), rows, cols, eps, _DTYPE[T], _stream(x)))
-    return res
-
-
-def gated_norm(o, g, w, eps):
-    """rmsnorm(o) * w * sigmoid(g); o [rows, cols], g [rows, cols] with any row stride."""
-    T = _type(o, "o")
-    _check(o, "o", T)
-    _check(g, "g", T, contiguous=False)
-    _check(w, "w", T)
-    if g.shape != o.shape or g.stride(1) != 1 or w.numel() != o.size(1):
-        raise RuntimeError("g must have the shape of o with contiguous rows, w one element per column")
-    out = torch.empty_like(o)
-    _lib.check_hybrid(_lib.load_hybrid().fah_gated_norm(_p(o), _p(g), g.stride(0), _p(w), _p(out), o.size(0), o.size(1), eps, _DTYPE[T],
-                                                        _stream(o)))
-    return out
-
-
-def clamped_glu(gu, limit, alpha, shift):
-    """gu [rows, 2n] = gate | linear branch: g sigmoid(alpha g) (u + shift) of the clamped branches."""
-    T = _type(gu, "gu")
-    _check(gu, "gu", T)
-    n = gu.size(1) // 2
-    out = torch.empty((gu.size(0), n), dtype=T, device=gu.device)
-    _lib.check_hybrid(_lib.load_hybrid().fah_clamped_glu(_p(gu), _p(out), gu.size(0), n, limit, alpha, shift, _DTYPE[T], _stream(gu)))
-    return out
-
-
-def side_gate(z, side, tokens, off):
-    """gelu_tanh(z) * side[tokens, off : off + n]; z [rows, n]."""
-    T = _type(z, "z")
-    _check(z, "z", T)
-    _check(side, "side", T)
-    _check(tokens, "tokens", torch.int64)
-    if tokens.numel() != z.size(0):
-        raise RuntimeError("tokens must have one entry per row")
-    out = torch.empty_like(z)
-    _lib.check_hybrid(_lib.load_hybrid().fah_side_gate(_p(z), _p(side), _p(tokens), side.size(0), side.size(1), off, _p(out), z.size(0),
-                                                       z.size(1), _DTYPE[T], _stream(z)))
-    return out
+def _check_rc(rc):
+    _lib.check(rc, "hybrid")
 
 
 def lightning(qkv, offsets, heads, dk, dv, decay, state, slots, starts, status, *, cu_seqlens=None, max_len=0):
@@ -128,10 +35,10 @@ def lightning(qkv, offsets, heads, dk, dv, decay, state, slots, starts, status, 
         raise RuntimeError("starts must have one entry per sequence")
     tokens = qkv.size(0)
     out = torch.empty((tokens, heads * dv), dtype=T, device=qkv.device)
-    lib, ws = _lib.load_hybrid(), None
+    lib, ws = _lib.library("hybrid"), None
     if cu_seqlens is not None:
         ws = _workspace(lib.fah_lightning_workspace(n_seq, heads, dk, dv, max_len, _DTYPE[T]), qkv.device)
-    _lib.check_hybrid(lib.fah_lightning(
+    _check_rc(lib.fah_lightning(
         _p(qkv), qkv.size(1), *offsets, heads, dk, dv, _p(decay), _p(state), state.size(0), _p(slots), _p(starts), _p(cu_seqlens), n_seq, max_len,
         tokens, _p(out), _p(ws), ws.numel() if ws is not None else 0, _p(status), _DTYPE[T], _stream(qkv)))
     return out
@@ -162,7 +69,7 @@ def latent_prep(down, off_q, q_rank, off_kv, kv_rank, off_r, rot_dim, wq, wkv, e
     new = lambda n: torch.empty((rows, n), dtype=T, device=down.device)
     cq = new(q_rank)
     c, r = (new(kv_rank), new(rot_dim)) if contiguous_kv else (None, None)
-    _lib.check_hybrid(_lib.load_hybrid().fah_latent_prep(
+    _check_rc(_lib.library("hybrid").fah_latent_prep(
         _p(down), down.size(1), off_q, q_rank, off_kv, kv_rank, off_r, rot_dim, _p(wq), _p(wkv), eps, _p(cos), _p(sin), _p(cq), _p(c), _p(r),
         _p(pool), pool.size(2), pool.size(0), _p(block_table), block_table.size(1), block_table.size(0), _p(tok_seq), _p(positions), rows,
         _p(status), _DTYPE[T], _stream(down)))
@@ -177,7 +84,7 @@ def rotate_heads_(q, cos, sin, heads, head_stride, off, rot_dim):
     _check(sin, "sin", torch.float32)
     if q.size(1) != heads * head_stride or cos.shape != (q.size(0), rot_dim // 2) or sin.shape != cos.shape:
         raise RuntimeError("q must be [rows, heads * head_stride], cos and sin [rows, rot_dim / 2]")
-    _lib.check_hybrid(_lib.load_hybrid().fah_rotate_heads(_p(q), _p(cos), _p(sin), q.size(0), heads, head_stride, off, rot_dim, _DTYPE[T],
+    _check_rc(_lib.library("hybrid").fah_rotate_heads(_p(q), _p(cos), _p(sin), q.size(0), heads, head_stride, off, rot_dim, _DTYPE[T],
                                                           _stream(q)))
     return q
 
@@ -200,9 +107,9 @@ def latent_attention(q_abs, q, q_off, cos, sin, pool, block_table, tok_seq, posi
         if gate.shape != (rows, heads) or gate.stride(1) != 1:
             raise RuntimeError("gate must be [rows, heads] with contiguous rows")
     out = torch.empty_like(q_abs)
-    lib = _lib.load_hybrid()
+    lib = _lib.library("hybrid")
     ws = _workspace(lib.fah_latent_attention_workspace(heads, kv_rank, rot_dim, rows, _DTYPE[T]), q_abs.device)
-    _lib.check_hybrid(lib.fah_latent_attention(
+    _check_rc(lib.fah_latent_attention(
         _p(q_abs), _p(q), q.size(2), q_off, _p(cos), _p(sin), _p(pool), pool.size(2), pool.size(0), _p(block_table), block_table.size(1),
         block_table.size(0), _p(tok_seq), _p(positions), _p(gate), gate.stride(0) if gate is not None else 0, heads, kv_rank, rot_dim, scale,
         _p(out), rows, _p(ws), ws.numel() if ws is not None else 0, _p(status), _DTYPE[T], _stream(q_abs)))
@@ -211,7 +118,7 @@ def latent_attention(q_abs, q, q_off, cos, sin, pool, block_table, tok_seq, posi
 
 def latent_prefill_supported(dim, rot_dim, vdim, scale, dtype):
     """Whether `latent_prefill` is built for these sizes."""
-    return dtype in _DTYPE and bool(_lib.load_hybrid().fah_latent_prefill_supported(dim, rot_dim, vdim, scale, _DTYPE[dtype]))
+    return dtype in _DTYPE and bool(_lib.library("hybrid").fah_latent_prefill_supported(dim, rot_dim, vdim, scale, _DTYPE[dtype]))
 
 
 def latent_prefill(q, kv, kr, gate, cu_q, cu_kv, max_q, heads, dim, vdim, scale, status):
@@ -231,7 +138,7 @@ def latent_prefill(q, kv, kr, gate, cu_q, cu_kv, max_q, heads, dim, vdim, scale,
         if gate.shape != (q.size(0), heads) or gate.stride(1) != 1:
             raise RuntimeError("gate must be [total_q, heads] with contiguous rows")
     out = torch.empty((q.size(0), heads * vdim), dtype=T, device=q.device)
-    _lib.check_hybrid(_lib.load_hybrid().fah_latent_prefill(
+    _check_rc(_lib.library("hybrid").fah_latent_prefill(
         _p(q), _p(kv), _p(kr), _p(gate), gate.stride(0) if gate is not None else 0, _p(cu_q), _p(cu_kv), cu_q.numel() - 1, max_q, q.size(0),
         kv.size(0), heads, dim, rot_dim, vdim, scale, _p(out), _p(status), _stream(q)))
     return out
@@ -247,7 +154,7 @@ def latent_gather(pool, block_table, cu_kv, total_kv, kv_rank, rot_dim, status):
         raise RuntimeError("cu_kv must have one entry more than block_table has rows")
     c = torch.empty((total_kv, kv_rank), dtype=T, device=pool.device)
     r = torch.empty((total_kv, rot_dim), dtype=T, device=pool.device)
-    _lib.check_hybrid(_lib.load_hybrid().fah_latent_gather(
+    _check_rc(_lib.library("hybrid").fah_latent_gather(
         _p(pool), pool.size(2), pool.size(0), _p(block_table), block_table.size(1), block_table.size(0), _p(cu_kv), total_kv, kv_rank, rot_dim,
         _p(c), _p(r), _p(status), _DTYPE[T], _stream(pool)))
     return c, r

@@ -131,8 +131,7 @@ class BlockManager:
         if total > len(self._tables[request_id]) * BLOCK_SIZE:
             raise ValueError("commit beyond the reserved blocks")
         self._tokens[request_id] = total
-        if self.sliding_window > 0 and total > self.sliding_window:
-            self._evict_sliding_window(request_id)
+        self._evict(request_id, self._first_needed(total))
 
     def release(self, request_id: str) -> None:
         """Return the request's blocks and its table row (manager.py:436-463).  A block shared with other
@@ -219,9 +218,13 @@ class BlockManager:
                 self._drop_ref(b)
 
     # ---- sliding window (manager.py:577-617) -------------------------------------------
-    def _evict_sliding_window(self, request_id: str) -> None:
-        """Give up the blocks whose tokens all lie before `length - sliding_window`."""
-        evictable_blocks = (self._tokens[request_id] - self.sliding_window) // BLOCK_SIZE      # (:588-596)
+    def _first_needed(self, total: int) -> int:
+        """Oldest position that a request with `total` tokens will still read."""
+        return max(total - self.sliding_window, 0) if self.sliding_window > 0 else 0
+
+    def _evict(self, request_id: str, first_needed: int) -> None:
+        """Give up the blocks whose tokens all lie before `first_needed`."""
+        evictable_blocks = min(first_needed // BLOCK_SIZE, len(self._tables[request_id]))      # (:588-596)
         done = self._evicted[request_id]
         if evictable_blocks <= done:
             return
@@ -302,28 +305,42 @@ class HybridCache(BlockManager):
     `specs` has one entry per layer run:
       ("latent", row)            a pool [num_blocks, 16, stride] of cached rows of `row` elements (stride: row rounded up
                                  to 16 bytes), addressed by the request's block table;
+      ("kv", heads, dim, vdim, chunk)   key and value pools [num_blocks, heads, 16, dim] and [num_blocks, heads, 16, vdim],
+                                 likewise; a token reads the keys of its chunk of `chunk` positions (0: all);
       ("state", heads, dk, dv)   a recurrent state [max_batch, heads, dk, dv] in fp32, one slot per request, addressed
-                                 by the request's table row.  A slot is not cleared when it changes hands: a request's
-                                 state starts at zero because the kernels take the state of position 0 as zero.
+                                 by the request's table row;
+      ("slots", (shape, dtype), ...)   a tuple of tensors [max_batch, *shape], likewise (dtype None: the model's).
+    A slot is not cleared when it changes hands: a request's state starts at zero because the kernels take the state of
+    position 0 as zero.
     The pages of a prefix do not bring back the recurrent state at its end, so prefixes are shared only by models
-    without one."""
+    without one.  When every layer that has pages reads only the current chunk, the blocks before it are given up."""
 
     def __init__(self, specs, num_blocks: int, max_batch: int, max_blocks_per_seq: int, device="cuda",
                  dtype=torch.bfloat16):
+        paged = [s for s in specs if s[0] in ("latent", "kv")]
+        self._chunks = {s[4] if s[0] == "kv" else 0 for s in paged}
         super().__init__(num_blocks, max_batch, max_blocks_per_seq, device,
-                         enable_prefix_cache=all(s[0] == "latent" for s in specs))
+                         enable_prefix_cache=len(paged) == len(specs) and not any(self._chunks))
         self.dtype = dtype
         align = 16 // torch.empty((), dtype=dtype).element_size()
+        zeros = lambda *shape, dtype=dtype: torch.zeros(shape, dtype=dtype, device=self.device)
         self.stores = []
         for spec in specs:
             if spec[0] == "latent":
                 stride = (spec[1] + align - 1) // align * align
-                self.stores.append(torch.zeros((num_blocks, BLOCK_SIZE, stride), dtype=dtype, device=self.device))
+                self.stores.append(zeros(num_blocks, BLOCK_SIZE, stride))
+            elif spec[0] == "kv":
+                self.stores.append(tuple(zeros(num_blocks, spec[1], BLOCK_SIZE, d) for d in spec[2:4]))
             elif spec[0] == "state":
-                self.stores.append(torch.zeros((max_batch,) + tuple(spec[1:]), dtype=torch.float32, device=self.device))
+                self.stores.append(zeros(max_batch, *spec[1:], dtype=torch.float32))
+            elif spec[0] == "slots":
+                self.stores.append(tuple(zeros(max_batch, *shape, dtype=dt or dtype) for shape, dt in spec[1:]))
             else:
                 raise ValueError(f"unknown store {spec[0]!r}")
         self.status = torch.zeros(1, dtype=torch.int32, device=self.device)     # written by the kernels
+
+    def _first_needed(self, total: int) -> int:
+        return min((total // c * c if c else 0 for c in self._chunks), default=total)
 
     def check_errors(self) -> None:
         st = int(self.status.item())

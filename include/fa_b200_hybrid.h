@@ -1,5 +1,5 @@
-/* C ABI of the hybrid decoder's operators (libfa_b200_hybrid.so, sm_100a): decayed linear attention, attention over
- * cached latent rows, and the row-wise operators between the matrix products.
+/* C ABI of the hybrid decoder's operators (libfa_b200_hybrid.so, sm_100a): decayed linear attention and attention over
+ * cached latent rows.  (The row-wise operators between the matrix products: fa_b200_rows.h.)
  *
  * Conventions: device pointers on the current device; every call is asynchronous on `stream` (a cudaStream_t);
  * nothing is allocated.  `dtype` is the type of activations, weights and cached latent rows: FAH_F32 or FAH_BF16; the
@@ -20,24 +20,6 @@ enum { FAH_F32 = 0, FAH_BF16 = 1 };
 enum { FAH_OK = 0, FAH_ERR_INVALID_ARGUMENT = -1, FAH_ERR_UNSUPPORTED = -2, FAH_ERR_CUDA = -4 };
 
 const char* fah_last_error(void);
-
-/* x [rows, cols] fp32: embed_mode 1 adds embed[token], 2 sets x to embed[token]; then delta [rows, cols] is added, RMS-normed
- * with weight delta_w first if that is given.  out [rows, cols] = rmsnorm(x) * w, or x itself if w is null; out may be null. */
-int fah_residual_norm(float* x, const void* delta, const void* delta_w, const void* embed, const int64_t* tokens,
-                      int embed_mode, int vocab, const void* w, void* out, int64_t rows, int cols, float eps, int dtype,
-                      void* stream);
-
-/* out [rows, cols] = rmsnorm(o [rows, cols]) * w * sigmoid(g), g with row stride g_stride. */
-int fah_gated_norm(const void* o, const void* g, int64_t g_stride, const void* w, void* out, int64_t rows, int cols, float eps,
-                   int dtype, void* stream);
-
-/* gu [rows, 2n]: out [rows, n] = g * sigmoid(alpha * g) * (u + shift), g = min(gu[:n], limit), u = clamp(gu[n:], -limit, limit). */
-int fah_clamped_glu(const void* gu, void* out, int64_t rows, int n, float limit, float alpha, float shift, int dtype,
-                    void* stream);
-
-/* out [rows, n] = gelu_tanh(z [rows, n]) * side[token, off : off + n], side with row stride side_stride. */
-int fah_side_gate(const void* z, const void* side, const int64_t* tokens, int vocab, int64_t side_stride, int off, void* out,
-                  int64_t rows, int n, int dtype, void* stream);
 
 /* Decayed linear attention with SiLU on q, k, v: per head S = decay * S + k v^T, o = S^T q.
  * qkv [tokens, stride] with the heads x dk queries at column off_q, keys at off_k, heads x dv values at off_v;

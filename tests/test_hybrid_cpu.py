@@ -58,7 +58,7 @@ def test_config_errors_are_refused(change):
 
 
 def test_registry_knows_both_families(tmp_path):
-    assert registry.architectures() == ["Berilix", "Qwen3"]
+    assert registry.architectures() == ["Berilix", "Qwen3", "Sabipel"]
     with pytest.raises(ValueError, match="unknown architecture"):
         registry.family_of({"architecture": "none"})
     fam = registry.family_of({"architecture": "Qwen3"})
@@ -224,25 +224,31 @@ def test_oracle_is_causal():
 
 
 # ---- library ---------------------------------------------------------------------------------------------------
-def test_hybrid_library_exports_every_declared_symbol():
+@pytest.mark.parametrize("library, prefix", [("rows", "far"), ("hybrid", "fah"), ("mixers", "fam")])
+def test_library_exports_every_declared_symbol(library, prefix):
     from flash_attn_v100_b200 import _lib
     from flash_attn_v100_b200.build import build
-    build(library="hybrid")
-    lib = _lib.load_hybrid()
-    text = re.sub(r"/\*.*?\*/", "", open(os.path.join(ROOT, "include", "fa_b200_hybrid.h")).read(), flags=re.S)
-    names = set(re.findall(r"\b(fah_[a-z0-9_]+)\s*\(", text))
-    assert names == set(_lib.HYBRID_SIGNATURES) and all(hasattr(lib, n) for n in names)
+    build(library=library)
+    lib = _lib.library(library)
+    text = re.sub(r"/\*.*?\*/", "", open(os.path.join(ROOT, "include", f"fa_b200_{library}.h")).read(), flags=re.S)
+    names = set(re.findall(rf"\b({prefix}_[a-z0-9_]+)\s*\(", text))
+    assert names == set(_lib._ABIS[library][0]) and all(hasattr(lib, n) for n in names)
 
 
-def test_hybrid_calls_check_their_arguments_before_the_device():
+def test_calls_check_their_arguments_before_the_device():
     from flash_attn_v100_b200 import _lib
-    lib = _lib.load_hybrid()
+    lib = _lib.library("rows")
     p = ctypes.c_void_p(256)
-    assert lib.fah_residual_norm(None, None, None, None, None, 0, 0, None, None, 1, 8, 1e-5, 1, None) == -1
-    assert b"x is null" in lib.fah_last_error()
-    assert lib.fah_residual_norm(p, None, None, None, None, 0, 0, None, None, 1, 8, 1e-5, 7, None) == -1
-    assert lib.fah_gated_norm(p, p, 4, p, p, 1, 8, 1e-5, 1, None) == -1
-    assert lib.fah_side_gate(p, p, p, 10, 8, 4, p, 1, 8, 1, None) == -1
+    norm = lambda **kw: lib.far_residual_norm(ctypes.byref(_lib.ResidualNorm(**dict(dict(rows=1, cols=8, eps=1e-5, dtype=1, embed_scale=1.0), **kw))), None)
+    assert norm() == -1
+    assert b"x is null" in lib.far_last_error()
+    assert norm(x=256, dtype=7) == -1
+    assert norm(x=256, w=256, out=256, w2=256) == -1 and norm(x=256, embed_scale=2.0) == -1
+    assert lib.far_gated_norm(p, p, 4, p, p, 8, 1, 8, 8, 0, 1e-5, 1, None) == -1
+    assert lib.far_gated_norm(p, p, 8, p, p, 8, 1, 8, 3, 0, 1e-5, 1, None) == -1
+    assert lib.far_side_gate(p, p, p, 10, 8, 4, p, 1, 8, 1, None) == -1
+    assert lib.far_bigram_rows(p, None, p, p, p, 1, 2, 1, 7, 3, 5, p, p, None) == -1
+    lib = _lib.library("hybrid")
     assert lib.fah_rotate_heads(p, p, p, 1, 2, 8, 4, 6, 1, None) == -1
     assert lib.fah_lightning(p, 10, 0, 4, 8, 2, 4, 4, p, p, 1, p, p, None, 1, 1, 1, p, None, 0, p, 1, None) == -1
     assert lib.fah_latent_prefill(p, p, p, None, 0, p, p, 1, 1, 1, 1, 2, 132, 64, 64, 0.1, p, p, None) == -2
