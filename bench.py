@@ -542,20 +542,21 @@ def run_engine(args):
 
 
 def run_hybrid(args):
-    """Prefill and decode throughput of the hybrid decoder beside the Qwen3-style decoder of equal size, and every kernel of
-    both beside its roofline (one GPU; see flash_attn_v100_b200/engine/hybrid_bench.py)."""
+    """Prefill and decode throughput of a hybrid decoder beside the closest others of equal size, and every kernel beside its
+    roofline (one GPU; see flash_attn_v100_b200/engine/hybrid_bench.py and sabipel_bench.py)."""
     device = torch.device("cuda", 0)
     torch.cuda.set_device(device)
-    from flash_attn_v100_b200.engine import hybrid_bench
+    import importlib
+    hybrid_bench = importlib.import_module(f"flash_attn_v100_b200.engine.{args.workload}_bench")
     peaks, peak_src = load_peaks()
     sampler = ClockSampler(0)
     sampler.start()
     kernels = hybrid_bench.kernel_records(device, args.steps, args.warmup, peaks, args.hybrid_kernel)
-    models = hybrid_bench.model_records(device, 3, 1) if args.hybrid_kernel == "all" else []
+    models = hybrid_bench.model_records(device, 3, 1) if args.hybrid_kernel in ("all", "models") else []
     clocks = sampler.stop()
     first = models[0] if models else {}
     print(json.dumps({
-        "metric": "hybrid_decoder_decode_tokens_per_s", "value": first.get("decode_tokens_per_s"), "unit": "tokens/s", "n_gpus": 1,
+        "metric": f"{args.workload}_decoder_decode_tokens_per_s", "value": first.get("decode_tokens_per_s"), "unit": "tokens/s", "n_gpus": 1,
         "steps": args.steps, "warmup": max(args.warmup, 3), "higher_is_better": True, "dtype": "bf16",
         "data": "synthetic (seeded random weights, uniform random token ids)", "models": models, "kernels": kernels,
         "peaks": {k: peaks[k] for k in ("hbm_gbs", "bf16_tflops")}, "peak_source": peak_src, "clocks": clocks,
@@ -910,8 +911,8 @@ def main():
     ap.add_argument("--steps", type=int, default=50)
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
-    ap.add_argument("--workload", default="paged_decode", choices=sorted(WORKLOADS) + ["engine", "hybrid"])
-    ap.add_argument("--hybrid-kernel", default="all", help="hybrid workload: time this kernel only")
+    ap.add_argument("--workload", default="paged_decode", choices=sorted(WORKLOADS) + ["engine", "hybrid", "sabipel"])
+    ap.add_argument("--hybrid-kernel", default="all", help="hybrid and sabipel workloads: time this kernel only ('models': no kernel)")
     ap.add_argument("--engine-tiny", action="store_true", help="engine workload on the tiny test shape")
     ap.add_argument("--engine-nccl-decode", action="store_true",
                     help="engine workload: NCCL collectives in the decode step (chain of CUDA graphs) instead of "
@@ -931,7 +932,7 @@ def main():
         run_reference(args)
     elif args.workload == "engine":
         run_engine(args)
-    elif args.workload == "hybrid":
+    elif args.workload in ("hybrid", "sabipel"):
         run_hybrid(args)
     else:
         run_b200(args)

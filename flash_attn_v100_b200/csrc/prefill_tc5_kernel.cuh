@@ -96,6 +96,13 @@ struct Tc5SharedParams : Tc5Params {
   long long gate_stride;
   int* status;               // caller's status word, beside g_prefill_status
 };
+// Builds with a distance bias.
+struct Tc5BiasParams : Tc5SharedParams {
+  const float* bias;         // [H_Q]: bias * (place of the key - place of the row) is added to the score before it is scaled
+  float inv_scale;           // what the biases are multiplied by to be that
+  const __nv_bfloat16* col_gate;   // output column c of head h times sigmoid(col_gate[r * col_gate_stride + h * D_real + c]) (null: not)
+  long long col_gate_stride;
+};
 
 __device__ __forceinline__ bool wait_or_abort(uint32_t bar, uint32_t parity, volatile int* abort_flag) {
   if (mbar_test_wait(bar, parity)) return true;  // cheap probe: the phase is usually complete already
@@ -291,18 +298,23 @@ __device__ __forceinline__ bool tc5_decode_item(const P& p, long long item, Tc5I
 // BF: q, k, v are bfloat16: the same kernel with bfloat16 MMA operands and P rounded to bfloat16.
 // Queries and keys are NA slabs of 64 columns from (qmap, kmap) followed by NB slabs from (qmap_b, kmap_b), whose keys all
 // heads share (NB = 0: the second maps are not used); values have D columns.
-template <int NA, int NB, int D, int NPOLY, bool BF>
+// BIAS: a distance bias on the scores and an element-wise gate on the output, packed sequences only.  In head-pair mode the KV tiles are
+// then walked from the diagonal backwards: the bias grows towards the diagonal, so the first tile has (nearly) every row's largest
+// score, where an ascending walk would raise the row's reference exponent at almost every tile.
+template <int NA, int NB, int D, int NPOLY, bool BF, bool BIAS = false>
 __global__ void __launch_bounds__(640, 1)
 prefill_tc5_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_constant__ CUtensorMap kmap,
                    const __grid_constant__ CUtensorMap vmap, const __grid_constant__ CUtensorMap qmap_b,
                    const __grid_constant__ CUtensorMap kmap_b,
-                   const std::conditional_t<(NB > 0), Tc5SharedParams, Tc5Params> p) {
+                   const std::conditional_t<BIAS, Tc5BiasParams, std::conditional_t<(NB > 0), Tc5SharedParams, Tc5Params>> p) {
   constexpr int BM = 128, BN = 128;
   using Layout = Tc5Layout<NA, NB, D>;
   constexpr int K_STAGES = Layout::K_STAGES, V_STAGES = Layout::V_STAGES;
   constexpr int SLAB = Layout::SLAB;         // bytes of a [128 rows][64 cols] 16-bit slab
   constexpr int NQK = NA + NB, NV = D / 64;
-  constexpr bool EXT = NB > 0;               // keys of earlier calls (cu_kv) and the head gates come with the shared-part builds
+  constexpr bool EXT = NB > 0 || BIAS;       // keys of earlier calls (cu_kv) and the head gates come with the shared-part builds
+  // KV tile of step j of an item with n steps
+  auto tile_of = [&](int j, int n) { return BIAS && p.pair_heads ? n - 1 - j : j; };
   constexpr int QK_BYTES = NQK * SLAB;       // one Q or K tile
   constexpr int V_BYTES = NV * SLAB;         // one V tile
   // instruction descriptor of kind::f16: fp32 accumulators (bit 4), operand formats (bits 7 and 10: 1 = bfloat16),
@@ -440,12 +452,12 @@ prefill_tc5_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_consta
 #pragma unroll
           for (int sl = 0; sl < NQK; ++sl)
             tma_load_3d(sK + st * QK_BYTES + sl * SLAB, sl < NA ? &kmap : &kmap_b, (sl < NA ? sl : sl - NA) * 64,
-                        sl < NA ? it.kv_c1 : 0, it.kv_c2 + j * BN, bar(B_KFULL + st));
+                        sl < NA ? it.kv_c1 : 0, it.kv_c2 + tile_of(j, it.n_max) * BN, bar(B_KFULL + st));
           if (kv_it >= V_STAGES) PROF_WAIT(0, 4, wait_or_abort(bar(B_VEMPTY + sv), phv ^ 1u, abort_flag));
           mbar_expect_tx(bar(B_VFULL + sv), V_BYTES);
 #pragma unroll
           for (int sl = 0; sl < NV; ++sl)
-            tma_load_3d(sV + sv * V_BYTES + sl * SLAB, &vmap, sl * 64, it.kv_c1, it.kv_c2 + j * BN, bar(B_VFULL + sv));
+            tma_load_3d(sV + sv * V_BYTES + sl * SLAB, &vmap, sl * 64, it.kv_c1, it.kv_c2 + tile_of(j, it.n_max) * BN, bar(B_VFULL + sv));
         }
       }
       // On the way out every copy issued above must have landed (on a regular exit they all have been
@@ -722,6 +734,19 @@ prefill_tc5_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_consta
       const int klen = EXT ? it.klen : it.len;
       const int grow = (EXT ? it.past : 0) + it.row0[t] + row;       // place of my row among the keys
       float m = 0.f, l = 0.f;
+      // BIAS: scores of chunk c get bias * (column inside the chunk) as they are read; the rest, the same for the whole chunk, goes to
+      // its maximum and to the exponent's offset.
+      const float bias = [&] { if constexpr (BIAS) return p.bias[it.head[t]] * p.inv_scale; else return 0.f; }();
+      auto add_bias = [&](float (&v)[32]) {
+        if constexpr (BIAS) {
+#pragma unroll
+          for (int i = 0; i < 16; ++i) {
+            const float2 r = ffma2(make_float2(bias, bias), make_float2((float)(2 * i), (float)(2 * i + 1)), make_float2(v[2 * i], v[2 * i + 1]));
+            v[2 * i] = r.x;
+            v[2 * i + 1] = r.y;
+          }
+        }
+      };
       for (int j = 0; j < n_mine; ++j, ++pph) {
         PROF_COUNT(3 + t, 14);
         PROF_WAIT(3 + t, 1, wait_or_abort(bar(B_SFULL + t), sph & 1u, abort_flag));
@@ -730,7 +755,8 @@ prefill_tc5_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_consta
         PROF_MARK(prof_t_s);
         tc_fence_after();
         forward_step(kv0, j, n_mine);
-        const int k0 = j * BN;
+        const int k0 = tile_of(j, n_mine) * BN;
+        auto chunk_bias = [&](int c) { return BIAS ? bias * (float)(k0 + c * 32 - grow) : 0.f; };
         const bool need_mask = (k0 + BN > klen) || (p.causal && (k0 + BN - 1 > (EXT ? it.past : 0) + it.row0[t]));
         // ---- my half of the score row: chunk c_lo (kept in registers) and chunk c_hi (read for its maximum,
         // read again when its turn comes).  Where P is written: thread 0 of the pair writes quarter 0 over
@@ -745,6 +771,7 @@ prefill_tc5_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_consta
           PROF_MARK(pf0);
           tc_ld32(tS + c_hi * 32, sw);
           tc_wait_ld();
+          add_bias(sw);
           PROF_MARK(pf1);
           float a0 = fmaxf(sw[0], sw[1]), a1 = fmaxf(sw[2], sw[3]);
 #pragma unroll
@@ -754,12 +781,14 @@ prefill_tc5_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_consta
           }
           tc_ld32(tS + c_lo * 32, sv);      // (one chunk in registers at a time: 104 registers per thread)
           tc_wait_ld();
+          add_bias(sv);
           PROF_MARK(pf2);
           lo_loaded = true;
           turn_wait(pph);
-          const float2 nm2 = make_float2(-m, -m);
-          exp_chunk_store<NPOLY, BF>(sv, sc2, nm2, rs_lo, tP + q_lo * 16);
-          const bool inside = (rs_lo.x + rs_lo.y <= 32768.f) && (fmaxf(a0, a1) * p.scale_log2 <= m + 15.f);   // false for NaN
+          const float nm_lo = BIAS ? fmaf(chunk_bias(c_lo), p.scale_log2, -m) : -m, nm_hi = BIAS ? fmaf(chunk_bias(c_hi), p.scale_log2, -m) : -m;
+          exp_chunk_store<NPOLY, BF>(sv, sc2, make_float2(nm_lo, nm_lo), rs_lo, tP + q_lo * 16);
+          const bool inside = (rs_lo.x + rs_lo.y <= 32768.f) &&
+                              ((BIAS ? fmaxf(a0, a1) + chunk_bias(c_hi) : fmaxf(a0, a1)) * p.scale_log2 <= m + 15.f);   // false for NaN
           const uint32_t tag = pph + 1u;
           if (__any_sync(0xffffffffu, !inside) && lane == 0) *my_tag = tag;
           PROF_MARK(pf3);
@@ -773,8 +802,9 @@ prefill_tc5_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_consta
             rs_lo = make_float2(0.f, 0.f);
           } else {
             tc_wait_ld();
+            add_bias(sw);
             PROF_MARK(pf6);
-            exp_chunk_store<NPOLY, BF>(sw, sc2, nm2, rs_hi, tP + q_hi * 16);
+            exp_chunk_store<NPOLY, BF>(sw, sc2, make_float2(nm_hi, nm_hi), rs_hi, tP + q_hi * 16);
             turn_pass();
             PROF_MARK(pf7);
             PROF_STAMP(2 + t);
@@ -819,14 +849,16 @@ prefill_tc5_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_consta
           };
           tc_ld32(tS + c_hi * 32, sw);
           tc_wait_ld();
+          add_bias(sw);
           mask_chunk(sw, c_hi);
-          const float mx_hi = max_chunk(sw);
+          const float mx_hi = max_chunk(sw) + (BIAS ? chunk_bias(c_hi) : 0.f);
           if (!lo_loaded) {
             tc_ld32(tS + c_lo * 32, sv);
             tc_wait_ld();
+            add_bias(sv);
           }
           mask_chunk(sv, c_lo);
-          const float mxl = fmaxf(mx_hi, max_chunk(sv));
+          const float mxl = fmaxf(mx_hi, max_chunk(sv) + (BIAS ? chunk_bias(c_lo) : 0.f));
           // the other half of the row lives in the partner warp
           float* slot_f = xch + (int)(pph & 1u) * (2 * 128);
           slot_f[h * 128 + row] = mxl;
@@ -851,14 +883,16 @@ prefill_tc5_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_consta
           l *= alpha;
           // ---- P = exp2(S * scale - m), fp16 ----
           const float neg_m = (m == -INFINITY) ? 0.f : -m;
-          const float2 nm2 = make_float2(neg_m, neg_m);
+          const float nm_lo = BIAS ? fmaf(chunk_bias(c_lo), p.scale_log2, neg_m) : neg_m;
+          const float nm_hi = BIAS ? fmaf(chunk_bias(c_hi), p.scale_log2, neg_m) : neg_m;
           if (!lo_loaded) turn_wait(pph);     // (a redone step has taken its turn already)
-          if (c_lo * 32 < lim_max) exp_chunk_store<NPOLY, BF>(sv, sc2, nm2, rs_lo, tP + q_lo * 16);
+          if (c_lo * 32 < lim_max) exp_chunk_store<NPOLY, BF>(sv, sc2, make_float2(nm_lo, nm_lo), rs_lo, tP + q_lo * 16);
           else zero_chunk_store(tP + q_lo * 16);
           tc_ld32(tS + c_hi * 32, sw);        // chunk c_hi again (its columns are written by nobody but me)
           tc_wait_ld();
+          add_bias(sw);
           mask_chunk(sw, c_hi);
-          if (c_hi * 32 < lim_max) exp_chunk_store<NPOLY, BF>(sw, sc2, nm2, rs_hi, tP + q_hi * 16);
+          if (c_hi * 32 < lim_max) exp_chunk_store<NPOLY, BF>(sw, sc2, make_float2(nm_hi, nm_hi), rs_hi, tP + q_hi * 16);
           else zero_chunk_store(tP + q_hi * 16);
           turn_pass();
           PROF_STAMP(2 + t);
@@ -929,6 +963,18 @@ prefill_tc5_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_consta
 #pragma unroll
       for (int k = 0; k < NU; ++k) {
         const int r = it.row0[t] + row_g + k;             // row within the sequence
+        if constexpr (BIAS) {
+          if (p.col_gate != nullptr && r < len && col < p.D_real) {
+            const uint4 g = *reinterpret_cast<const uint4*>(p.col_gate + (it.tok0 + r) * p.col_gate_stride + (long long)it.head[t] * p.D_real + col);
+            const uint32_t gw[4] = {g.x, g.y, g.z, g.w};
+#pragma unroll
+            for (int w = 0; w < 4; ++w) {
+              const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gw[w]));
+              const float2 o = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u[k][w]));
+              u[k][w] = pack_bf162(__fdividef(o.x, 1.f + __expf(-z.x)), __fdividef(o.y, 1.f + __expf(-z.y)));
+            }
+          }
+        }
         if (r < len && col < p.D_real)
           *reinterpret_cast<uint4*>(obase + (long long)r * p.o_tok_stride + col) = make_uint4(u[k][0], u[k][1], u[k][2], u[k][3]);
       }

@@ -213,9 +213,9 @@ class HybridConfig:
             self.bigram.validate()
         if self.loop_times > 1 and (self.bigram is not None or self.max_positions or self.embed_scale != 1.0):
             raise ValueError("a loop adds the plain token embeddings again: it does not go with a scaled or summed embedding")
-        values = {(l.mixer.kv_heads, l.mixer.vdim) for l in self.layers if isinstance(l.mixer, ChunkedAttentionSpec) and l.mixer.v_mix}
+        values = {l.mixer.kv_heads * l.mixer.vdim for l in self.layers if isinstance(l.mixer, ChunkedAttentionSpec) and l.mixer.v_mix}
         if len(values) > 1:
-            raise ValueError(f"layers that mix values must have the same value heads, got {sorted(values)}")
+            raise ValueError(f"layers that mix values must have values of the same size, got {sorted(values)}")
 
     def runs(self) -> List[Tuple[int, bool]]:
         """(layer index, add the embedding output first) of every layer run, in order."""

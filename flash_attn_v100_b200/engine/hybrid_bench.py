@@ -172,13 +172,15 @@ def kernel_records(device, steps, warmup, peaks, which="all"):
     return out
 
 
-def model_records(device, steps, warmup):
-    """Prefill and decode throughput of both models through `GenerationRunner.generate`."""
+def model_records(device, steps, warmup, hybrids=None):
+    """Prefill and decode throughput of the hybrid decoders (name -> configuration) and of the Qwen3-style decoder through
+    `GenerationRunner.generate`."""
     out = []
     shapes = ((256, 1024, 64, 16), (64, 4096, 64, 4), (8, 8192, 64, 2))
-    for name in ("hybrid", "qwen3"):
-        if name == "hybrid":
-            cfg = hybrid_config()
+    hybrids = hybrids or {"hybrid": hybrid_config()}
+    for name in (*hybrids, "qwen3"):
+        if name in hybrids:
+            cfg = hybrids[name]
             model = HybridDecoder(cfg, hybrid_weights(cfg, random_hybrid_tensors(cfg, 0, device), torch.bfloat16, device), device)
         else:
             cfg = qwen_config()
