@@ -82,7 +82,9 @@ int fam_recurrence(const FamRecurrence* p, void* stream) {
     a.seg_state = static_cast<float*>(p->workspace);
     a.seg_norm = need ? a.seg_state + n * a.dk * a.dv : nullptr;
     a.seg_log = need ? a.seg_norm + n * a.dk : nullptr;
-    return done(mx::launch_recurrence_tc5(a, st(stream)), "recurrence_tc5");
+    void* enc = tensor_map_encode();
+    if (enc == nullptr) return fail(FAM_ERR_CUDA, "cuTensorMapEncodeTiled is not available from the driver");
+    return done(mx::launch_recurrence_tc5(a, enc, st(stream)), "recurrence_tc5");
   }
   return done(FAM_DISPATCH(p->dtype, mx::launch_recurrence_scan, a, st(stream)), "recurrence_scan");
 }

@@ -109,10 +109,10 @@ bool recurrence_step_supported(const RecurrenceArgs& a);
 template <typename T> cudaError_t launch_max_gate_step(const MaxGateStepArgs& a, int sm_count, cudaStream_t s);
 template <typename T> cudaError_t launch_ssd_step(const SsdStepArgs& a, int sm_count, cudaStream_t s);
 
-// Prompts in chunks on the tensor cores (bfloat16; dk <= 128, dk and dv multiples of 8).
+// Prompts in chunks on the tensor cores (bfloat16; dk <= 128, dk and dv multiples of 8).  `encode_fn` is cuTensorMapEncodeTiled.
 int recurrence_segments(int n_seq, int heads, int kv_rep, int dk, int dv, int max_len, int sm_count, int* seg_len);
 bool recurrence_tc5_supported(const RecurrenceArgs& a);
-cudaError_t launch_recurrence_tc5(const RecurrenceArgs& a, cudaStream_t s);
+cudaError_t launch_recurrence_tc5(const RecurrenceArgs& a, void* encode_fn, cudaStream_t s);
 
 }  // namespace mixers
 }  // namespace fa

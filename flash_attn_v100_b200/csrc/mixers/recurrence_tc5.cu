@@ -16,11 +16,13 @@
 // at the start of each, and the main launch then runs all segments side by side.
 //
 // Tensor memory, 512 columns: A / P of the first head [0, 128)  O1 [128, 256)  O2 [256, 384)  P of the second head / dS [384, 512).
-// Shared memory: five tiles of 128 x 128 bfloat16 (Q, K, V, and S high and low, whose place V' takes once O1 is done), each two
-// 128-byte-swizzled slabs of 64 columns.  Waits are bounded: one that runs out sets the status word and the CTA leaves after another
-// bounded wait for its MMAs.
+// Shared memory: six tiles of 128 x 128 bfloat16, each two 128-byte-swizzled slabs of 64 columns: Q, K twice, V, and S high and low,
+// whose place V' takes once O1 is done.  Q, K and V come by TMA (the next K while this chunk is computed, the next Q once O1 is done,
+// the next V once the output, which takes V's place, has been stored, also by TMA).  Rows past a sequence's end have the weight 0.
+// Waits are bounded: one that runs out sets the status word and the CTA leaves after another bounded wait for its MMAs and copies.
 #include "../hybrid/hybrid_common.cuh"
 #include "../tc5.cuh"
+#include "../tma3.cuh"
 #include "recurrence.cuh"
 
 namespace fa {
@@ -44,10 +46,11 @@ struct Small {                 // behind the tiles
   float n[N];                  // normaliser
   float n_add[kThreads / 32][N];
   float den[4][C];             // partial n . q of every row, by column group
-  uint64_t bars[4];
+  uint64_t bars[8];
   uint32_t tmem_slot;
 };
-constexpr int kSmem = 1024 + 5 * TILE + (int)sizeof(Small);
+constexpr int kTiles = 6;
+constexpr int kSmem = 1024 + kTiles * TILE + (int)sizeof(Small);
 static_assert(kSmem <= 227 * 1024, "shared memory plan exceeds the SM");
 
 // Byte offset of 16-byte unit `u` (0..15) of row `row` in a tile.
@@ -66,14 +69,16 @@ __device__ __forceinline__ float2 unpack2(uint32_t v) {
   return make_float2(__uint_as_float(v << 16), __uint_as_float(v & 0xffff0000u));
 }
 // Two fp32 numbers as packed (high, low) bfloat16 parts.
-__device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
-  hi = pack_bf162(x, y);
-  const float2 r = unpack2(hi);
-  lo = pack_bf162(x - r.x, y - r.y);
+__device__ __forceinline__ void split2(float2 v, uint32_t& hi, uint32_t& lo) {
+  hi = pack_bf162(v.x, v.y);
+  const float2 r = ffma2(unpack2(hi), make_float2(-1.f, -1.f), v);
+  lo = pack_bf162(r.x, r.y);
 }
 
 template <bool STATE_ONLY, int NH, bool NORM>
-__global__ void __launch_bounds__(kThreads, 1) recurrence_tc5_kernel(const RecurrenceArgs a) {
+__global__ void __launch_bounds__(kThreads, 1)
+recurrence_tc5_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_constant__ CUtensorMap kmap, const __grid_constant__ CUtensorMap vmap,
+                      const __grid_constant__ CUtensorMap omap, const RecurrenceArgs a) {
   static_assert(NH == 1 || !NORM, "a pair of heads has no normaliser");
   // instruction descriptors: fp32 accumulators, bfloat16 operands, M = 128, N at bit 17; bit 15: A MN-major, bit 16: B MN-major
   constexpr uint32_t IDESC = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(128 >> 4) << 24);
@@ -83,9 +88,10 @@ __global__ void __launch_bounds__(kThreads, 1) recurrence_tc5_kernel(const Recur
   extern __shared__ uint8_t smem_dyn[];
   const uint32_t raw_base = smem_u32(smem_dyn);
   uint8_t* smem = smem_dyn + ((1024u - (raw_base & 1023u)) & 1023u);
-  const uint32_t sQ = smem_u32(smem), sK = sQ + TILE, sV = sK + TILE, sSh = sV + TILE, sSl = sSh + TILE;
-  Small& sm = *reinterpret_cast<Small*>(smem + 5 * TILE);
-  const uint32_t bar_a = smem_u32(&sm.bars[0]), bar_1 = smem_u32(&sm.bars[1]), bar_o = smem_u32(&sm.bars[2]), bar_s = smem_u32(&sm.bars[3]);
+  const uint32_t sQ = smem_u32(smem), sK0 = sQ + TILE, sV = sK0 + 2 * TILE, sSh = sV + TILE, sSl = sSh + TILE;
+  Small& sm = *reinterpret_cast<Small*>(smem + kTiles * TILE);
+  auto bar = [&](int i) { return smem_u32(&sm.bars[i]); };
+  const uint32_t bar_a = bar(0), bar_1 = bar(1), bar_o = bar(2), bar_s = bar(3), full_q = bar(4), full_v = bar(5), full_k = bar(6);   // full_k: two
 
   const int seq = blockIdx.x / a.max_segs, seg = blockIdx.x - seq * a.max_segs;
   const int head0 = blockIdx.y * NH, c0 = blockIdx.z * N, grp = head0 / a.kv_rep;
@@ -109,9 +115,30 @@ __global__ void __launch_bounds__(kThreads, 1) recurrence_tc5_kernel(const Recur
   const bool segmented = a.max_segs > 1;
   const long long seg_at = ((long long)seq * a.max_segs + seg) * a.heads;      // + head
 
-  if (tid == 0) {
-    for (int i = 0; i < 4; ++i) mbar_init(smem_u32(&sm.bars[i]), 1);
+  // ---- copies: one thread issues them all ------------------------------------------------------------
+  const bool copier = tid == kThreads - 32;
+  const bool wide_k = a.dk > 64, wide_v = NH == 2 || a.dv - c0 > 64;           // the tile's second slab has columns
+  auto load_tile = [&](const CUtensorMap* map, uint32_t dst, uint32_t full, bool wide, int col, int head, int col2, int head2, long long t) {
+    mbar_expect_tx(full, wide ? TILE : SLAB);
+    tma_load_3d(dst, map, col, head, (int)t, full);
+    if (wide) tma_load_3d(dst + SLAB, map, col2, head2, (int)t, full);
+  };
+  auto load_q = [&](int chunk) { load_tile(&qmap, sQ, full_q, wide_k, 0, grp, 64, grp, t0 + (long long)chunk * C); };
+  auto load_k = [&](int chunk) {
+    load_tile(&kmap, sK0 + (chunk & 1) * TILE, full_k + (chunk & 1) * 8, wide_k, 0, grp, 64, grp, t0 + (long long)chunk * C);
+  };
+  auto load_v = [&](int chunk) {
+    if (NH == 2) load_tile(&vmap, sV, full_v, true, 0, head0, 0, head0 + 1, t0 + (long long)chunk * C);
+    else load_tile(&vmap, sV, full_v, wide_v, c0, head0, c0 + 64, head0, t0 + (long long)chunk * C);
+  };
+  int n_q = 0, n_k = 0, n_v = 0;                   // (copier) loads issued
+  if (copier) {
+    for (int i = 0; i < 8; ++i) mbar_init(bar(i), 1);
     mbar_fence_init();
+    fence_proxy_async();
+    if (!STATE_ONLY) { load_q(0); ++n_q; }
+    load_k(0); ++n_k;
+    load_v(0); ++n_v;
   }
   if (warp == 0) {
     asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&sm.tmem_slot)), "r"(512u) : "memory");
@@ -125,11 +152,13 @@ __global__ void __launch_bounds__(kThreads, 1) recurrence_tc5_kernel(const Recur
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const bool in = tb + i < t1;
-      gl[i] = in ? a.la[at + i] * kLog2e : 0.f;
+      gl[i] = in ? a.la[at + i] : 0.f;
       gb[i] = in ? a.b[at + i] : 0.f;
     }
   };
   auto put_gates = [&](int buf) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) gl[i] *= kLog2e;
     float up = gl[0] + gl[1] + gl[2] + gl[3], down = up;       // sums up to my last token, and from my first token on
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
@@ -162,6 +191,18 @@ __global__ void __launch_bounds__(kThreads, 1) recurrence_tc5_kernel(const Recur
       v = segmented ? a.seg_norm[(seg_at + head0) * a.dk + tid] : a.n0[((long long)seq * a.heads + head0) * a.dk + tid];
     sm.n[tid] = v;
   }
+  if (!wide_k || !wide_v) {                                    // slabs that no copy fills
+    const uint4 z = make_uint4(0, 0, 0, 0);
+    for (int i = tid; i < SLAB / 16; i += kThreads) {
+      if (!wide_k) {
+        st_shared(sQ + SLAB + i * 16, z);
+        st_shared(sK0 + SLAB + i * 16, z);
+        st_shared(sK0 + TILE + SLAB + i * 16, z);
+      }
+      if (!wide_v) st_shared(sV + SLAB + i * 16, z);
+    }
+    fence_proxy_async();
+  }
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
@@ -193,120 +234,66 @@ __global__ void __launch_bounds__(kThreads, 1) recurrence_tc5_kernel(const Recur
     }
   }
 
-  // ---- fetching: four 16-byte units of each of q, k and v per thread --------------------------------
-  const bf16* base = static_cast<const bf16*>(a.qkv);
-  const int cu8 = (tid & 15) * 8, urow = tid >> 4;           // unit n of mine: row urow + 32 n, columns cu8 .. + 7
+  // 16-byte unit n of mine where tiles are worked on row by row: row urow + 32 n, unit tid & 15
+  const int cu8 = (tid & 15) * 8, urow = tid >> 4;
   const int uh = NH == 2 ? cu8 >> 6 : 0, uc = NH == 2 ? cu8 & 63 : c0 + cu8;     // as value columns: a head and its columns
-  const bool k_ok = cu8 < a.dk, v_ok = uc < a.dv;
-  const int v_col = (head0 + uh) * a.dv + uc;
-  uint4 rq[STATE_ONLY ? 1 : 4], rk[4], rv[4];
-  auto fetch = [&](int chunk) {
-    const long long tb = t0 + (long long)chunk * C + urow;
-    const bf16* p = base + tb * a.stride;
-#pragma unroll
-    for (int n = 0; n < 4; ++n) {
-      const bool in = tb + 32 * n < t1;
-      const bf16* pr = p + (long long)(32 * n) * a.stride;
-      const uint4 z = make_uint4(0, 0, 0, 0);
-      if (!STATE_ONLY) rq[n] = in && k_ok ? *reinterpret_cast<const uint4*>(pr + a.off_q + grp * a.dk + cu8) : z;
-      rk[n] = in && k_ok ? *reinterpret_cast<const uint4*>(pr + a.off_k + grp * a.dk + cu8) : z;
-      rv[n] = in && v_ok ? *reinterpret_cast<const uint4*>(pr + a.off_v + v_col) : z;
-    }
-  };
-  // the rows that fetch() will read, on their way to the L2 while the current chunk is computed
-  auto prefetch = [&](int chunk) {
-    const long long tb = t0 + (long long)chunk * C + urow;
-#pragma unroll
-    for (int n = 0; n < 4; ++n) {
-      if (tb + 32 * n < t1 && (tid & 7) == 0) {
-        const bf16* pr = base + (tb + 32 * n) * a.stride;
-        if (!STATE_ONLY && k_ok) asm volatile("prefetch.global.L2 [%0];" ::"l"(pr + a.off_q + grp * a.dk + cu8));
-        if (k_ok) asm volatile("prefetch.global.L2 [%0];" ::"l"(pr + a.off_k + grp * a.dk + cu8));
-        if (v_ok) asm volatile("prefetch.global.L2 [%0];" ::"l"(pr + a.off_v + v_col));
-      }
-    }
-  };
-  // The finished chunk's output lies in the Q tile; every thread stores the units it will overwrite with the next queries.
-  auto store_out = [&](int done) {
-    const long long tb = t0 + (long long)done * C + urow;
-    bf16* p = static_cast<bf16*>(a.out) + tb * ((long long)a.heads * a.dv) + v_col;
-#pragma unroll
-    for (int n = 0; n < 4; ++n) {
-      const uint4 v = ld_shared(sQ + tile_off(urow + 32 * n, tid & 15));
-      if (v_ok && tb + 32 * n < t1) *reinterpret_cast<uint4*>(p + (long long)(32 * n) * a.heads * a.dv) = v;
-    }
-  };
 
   const float skip = a.skip != nullptr ? a.skip[head0 + mh] : 0.f;
   float log_sum = 0.f;                                        // (STATE_ONLY) log2 decay over the segment
   bool ok = true;
   uint32_t phase = 0;
-  fetch(0);
   int chunk = 0;
   for (; chunk < n_chunk; ++chunk, phase ^= 1u) {
     const int buf = chunk & 1;
-    if (chunk + 1 < n_chunk) prefetch(chunk + 1);
-    if (!STATE_ONLY && chunk > 0) store_out(chunk - 1);
-    // ---- tiles ----------------------------------------------------------------------------------------
-    if constexpr (NORM) {                                     // what the chunk adds to n
-      float add[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    const bool more = chunk + 1 < n_chunk;
+    const uint32_t sK = sK0 + (uint32_t)buf * TILE;
+    const uint32_t kphase = (uint32_t)(chunk >> 1) & 1u;
+    auto k_full = [&] { return mbar_wait(full_k + (uint32_t)buf * 8u, kphase); };
+
+    // v' = weight * v of the units of mine, high and low part, to the state's tiles
+    auto put_weighted = [&]() {
 #pragma unroll
       for (int n = 0; n < 4; ++n) {
-        const float w = sm.wk[buf][0][urow + 32 * n];
-        const uint32_t k[4] = {rk[n].x, rk[n].y, rk[n].z, rk[n].w};
-#pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const float2 f = unpack2(k[i]);
-          add[2 * i] += w * f.x;
-          add[2 * i + 1] += w * f.y;
-        }
+        const uint32_t off = tile_off(urow + 32 * n, tid & 15);
+        const float w1 = sm.wk[buf][uh][urow + 32 * n];
+        const float2 w = make_float2(w1, w1);
+        const uint4 v = ld_shared(sV + off);
+        uint4 h, l;
+        split2(fmul2(unpack2(v.x), w), h.x, l.x);
+        split2(fmul2(unpack2(v.y), w), h.y, l.y);
+        split2(fmul2(unpack2(v.z), w), h.z, l.z);
+        split2(fmul2(unpack2(v.w), w), h.w, l.w);
+        st_shared(sSh + off, h);
+        st_shared(sSl + off, l);
       }
-#pragma unroll
-      for (int i = 0; i < 8; ++i) add[i] += __shfl_xor_sync(0xffffffffu, add[i], 16);
-      if (lane < 16) {
-#pragma unroll
-        for (int i = 0; i < 8; ++i) sm.n_add[warp][cu8 + i] = add[i];
-      }
-    }
-    // v' of a unit, high and low part
-    auto weighted = [&](const uint4& v, int r, uint4& h, uint4& l) {
-      const float w = sm.wk[buf][uh][r];
-      float2 f;
-      f = unpack2(v.x); split2(f.x * w, f.y * w, h.x, l.x);
-      f = unpack2(v.y); split2(f.x * w, f.y * w, h.y, l.y);
-      f = unpack2(v.z); split2(f.x * w, f.y * w, h.z, l.z);
-      f = unpack2(v.w); split2(f.x * w, f.y * w, h.w, l.w);
     };
+    auto put_norm_sums = [&]() {                              // what the chunk adds to n, by warp
+      float2 add[4] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f), make_float2(0.f, 0.f), make_float2(0.f, 0.f)};
 #pragma unroll
-    for (int n = 0; n < 4; ++n) {
-      const uint32_t off = tile_off(urow + 32 * n, tid & 15);
-      st_shared(sK + off, rk[n]);
-      if constexpr (!STATE_ONLY) {
-        st_shared(sQ + off, rq[n]);
-        st_shared(sV + off, rv[n]);
-      } else {
-        uint4 h, l;
-        weighted(rv[n], urow + 32 * n, h, l);
-        st_shared(sSh + off, h);
-        st_shared(sSl + off, l);
+      for (int n = 0; n < 4; ++n) {
+        const float w1 = sm.wk[buf][0][urow + 32 * n];
+        const float2 w = make_float2(w1, w1);
+        const uint4 k = ld_shared(sK + tile_off(urow + 32 * n, tid & 15));
+        add[0] = ffma2(unpack2(k.x), w, add[0]);
+        add[1] = ffma2(unpack2(k.y), w, add[1]);
+        add[2] = ffma2(unpack2(k.z), w, add[2]);
+        add[3] = ffma2(unpack2(k.w), w, add[3]);
       }
-    }
-    if constexpr (!STATE_ONLY) {
 #pragma unroll
-      for (int u = 0; u < 4; ++u) {
-        uint4 h, l;
-        split2(S[8 * u], S[8 * u + 1], h.x, l.x);
-        split2(S[8 * u + 2], S[8 * u + 3], h.y, l.y);
-        split2(S[8 * u + 4], S[8 * u + 5], h.z, l.z);
-        split2(S[8 * u + 6], S[8 * u + 7], h.w, l.w);
-        const uint32_t off = tile_off(row, cg * 4 + u);
-        st_shared(sSh + off, h);
-        st_shared(sSl + off, l);
+      for (int i = 0; i < 4; ++i) {
+        add[i].x += __shfl_xor_sync(0xffffffffu, add[i].x, 16);
+        add[i].y += __shfl_xor_sync(0xffffffffu, add[i].y, 16);
+        if (lane < 16) *reinterpret_cast<float2*>(&sm.n_add[warp][cu8 + 2 * i]) = add[i];
       }
-    }
-    fence_proxy_async();
-    tc_fence_before();                                        // the last chunk's tensor-memory reads are done
-    __syncthreads();
+    };
+    auto advance_norm = [&]() {
+      if (tid < N) {
+        float v = sm.n[tid] * fast_exp2(sm.dec[buf][0]);
+#pragma unroll
+        for (int w = 0; w < kThreads / 32; ++w) v += sm.n_add[w][tid];
+        sm.n[tid] = v;
+      }
+    };
     const uint64_t khd = smem_desc(sK, SLAB, 1024), shd = smem_desc(sSh, SLAB, 1024), sld = smem_desc(sSl, SLAB, 1024);
     auto issue_state = [&]() {
 #pragma unroll
@@ -316,7 +303,32 @@ __global__ void __launch_bounds__(kThreads, 1) recurrence_tc5_kernel(const Recur
       }
       tc_commit(bar_s);
     };
+
+    // ---- the state's tiles: S, or (STATE_ONLY) V' at once ------------------------------------------------
+    if constexpr (STATE_ONLY) {
+      ok = mbar_wait(full_v, phase) && ok;
+      ok = k_full() && ok;
+      put_weighted();
+      if constexpr (NORM) put_norm_sums();
+    } else {
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        uint4 h, l;
+        split2(make_float2(S[8 * u], S[8 * u + 1]), h.x, l.x);
+        split2(make_float2(S[8 * u + 2], S[8 * u + 3]), h.y, l.y);
+        split2(make_float2(S[8 * u + 4], S[8 * u + 5]), h.z, l.z);
+        split2(make_float2(S[8 * u + 6], S[8 * u + 7]), h.w, l.w);
+        const uint32_t off = tile_off(row, cg * 4 + u);
+        st_shared(sSh + off, h);
+        st_shared(sSl + off, l);
+      }
+    }
+    fence_proxy_async();
+    tc_fence_before();                                        // the last chunk's tensor-memory reads are done
+    __syncthreads();
     if (warp == 0) {
+      if constexpr (!STATE_ONLY) ok = mbar_wait(full_q, phase) && ok;
+      ok = k_full() && ok;
       tc_fence_after();
       __syncwarp();
       if constexpr (STATE_ONLY) {
@@ -338,23 +350,36 @@ __global__ void __launch_bounds__(kThreads, 1) recurrence_tc5_kernel(const Recur
         tc_commit(bar_1);
       }
     }
-    if (warp < NH && chunk + 1 < n_chunk) fetch_gates(chunk + 1);
+    if (copier) {
+      if (more) { load_k(chunk + 1); ++n_k; }                 // (its last readers were done before the last chunk's end)
+      if (!STATE_ONLY && chunk > 0) {                         // the output has left V's place
+        tma_store_wait_read();
+        load_v(chunk);
+        ++n_v;
+      }
+      if (STATE_ONLY && more) { load_v(chunk + 1); ++n_v; }   // V has become V'
+    }
+    __syncwarp();
+    if (warp < NH && more) fetch_gates(chunk + 1);
     if constexpr (!STATE_ONLY) {
       float floor = 0.f, den = 0.f;
       if constexpr (NORM) {
         const long long t = t0 + (long long)chunk * C + row;
         if (t < t1) floor = a.floor[(long long)head0 * a.total + t];
+        ok = mbar_wait(full_q, phase) && ok;
+        ok = k_full() && ok;
+        put_norm_sums();
+        float2 d2 = make_float2(0.f, 0.f);
 #pragma unroll
         for (int u = 0; u < 4; ++u) {
           const uint4 q = ld_shared(sQ + tile_off(row, cg * 4 + u));
-          const float* n = sm.n + cg * 32 + u * 8;
-          float2 f;
-          f = unpack2(q.x); den += f.x * n[0] + f.y * n[1];
-          f = unpack2(q.y); den += f.x * n[2] + f.y * n[3];
-          f = unpack2(q.z); den += f.x * n[4] + f.y * n[5];
-          f = unpack2(q.w); den += f.x * n[6] + f.y * n[7];
+          const float4 n0 = *reinterpret_cast<const float4*>(sm.n + cg * 32 + u * 8), n1 = *reinterpret_cast<const float4*>(sm.n + cg * 32 + u * 8 + 4);
+          d2 = ffma2(unpack2(q.x), make_float2(n0.x, n0.y), d2);
+          d2 = ffma2(unpack2(q.y), make_float2(n0.z, n0.w), d2);
+          d2 = ffma2(unpack2(q.z), make_float2(n1.x, n1.y), d2);
+          d2 = ffma2(unpack2(q.w), make_float2(n1.z, n1.w), d2);
         }
-        den *= fast_exp2(sm.lb[buf][0][row].x);
+        den = (d2.x + d2.y) * fast_exp2(sm.lb[buf][0][row].x);
       }
       // ---- A -> P ------------------------------------------------------------------------------------
       ok = mbar_wait(bar_a, phase) && ok;
@@ -365,15 +390,9 @@ __global__ void __launch_bounds__(kThreads, 1) recurrence_tc5_kernel(const Recur
       tc_fence_before();
       __syncthreads();                                        // P is written over other warps' part of A; n has been read
       tc_fence_after();
-      if constexpr (NORM) {
-        if (tid < N) {
-          float v = sm.n[tid] * fast_exp2(sm.dec[buf][0]);
-#pragma unroll
-          for (int w = 0; w < kThreads / 32; ++w) v += sm.n_add[w][tid];
-          sm.n[tid] = v;
-        }
-      }
-      const bool below = cg * 32 <= (warp & 3) * 32 + 31;     // some of my columns are at or before some of my rows
+      if constexpr (NORM) advance_norm();
+      const int over = row - cg * 32;                         // my columns up to this one are at or before my row
+      const bool below = __any_sync(0xffffffffu, over >= 0);
 #pragma unroll
       for (int hh = 0; hh < NH; ++hh) {
         const float2* lb = sm.lb[buf][hh] + cg * 32;
@@ -381,17 +400,21 @@ __global__ void __launch_bounds__(kThreads, 1) recurrence_tc5_kernel(const Recur
 #pragma unroll
         for (int h = 0; h < 2; ++h) {
           uint32_t ph[8], pl[8];
+          if (below) {
 #pragma unroll
-          for (int i = 0; i < 8; ++i) {
-            const int j = h * 16 + 2 * i;
-            float x = 0.f, y = 0.f;
-            if (below) {
+            for (int i = 0; i < 8; ++i) {
+              const int j = h * 16 + 2 * i;
               const float4 w = *reinterpret_cast<const float4*>(lb + j);
-              if (cg * 32 + j <= row) x = s[j] * (w.y * fast_exp2(li - w.x));
-              if (cg * 32 + j + 1 <= row) y = s[j + 1] * (w.w * fast_exp2(li - w.z));
+              const float2 e = make_float2(fast_exp2(li - w.x), fast_exp2(li - w.z));
+              float2 p = fmul2(make_float2(s[j], s[j + 1]), fmul2(e, make_float2(w.y, w.w)));
+              p.x = j <= over ? p.x : 0.f;                    // (a selection: what is dropped may have overflowed)
+              p.y = j + 1 <= over ? p.y : 0.f;
+              if constexpr (NORM) den += p.x + p.y;
+              split2(p, ph[i], pl[i]);
             }
-            if constexpr (NORM) den += x + y;
-            split2(x, y, ph[i], pl[i]);
+          } else {
+#pragma unroll
+            for (int i = 0; i < 8; ++i) ph[i] = pl[i] = 0u;
           }
           tc_st8(tP + hh * 384u + h * 8u, ph);
           tc_st8(tP + hh * 384u + 64u + h * 8u, pl);
@@ -402,6 +425,7 @@ __global__ void __launch_bounds__(kThreads, 1) recurrence_tc5_kernel(const Recur
       tc_fence_before();
       __syncthreads();
       if (warp == 0) {
+        ok = mbar_wait(full_v, phase) && ok;
         tc_fence_after();
         __syncwarp();
         const uint64_t vd = smem_desc(sV, SLAB, 1024);
@@ -419,26 +443,18 @@ __global__ void __launch_bounds__(kThreads, 1) recurrence_tc5_kernel(const Recur
       }
       // ---- V' over the state's tiles ----------------------------------------------------------------
       ok = mbar_wait(bar_1, phase) && ok;
-#pragma unroll
-      for (int n = 0; n < 4; ++n) {
-        const uint32_t off = tile_off(urow + 32 * n, tid & 15);
-        uint4 h, l;
-        weighted(ld_shared(sV + off), urow + 32 * n, h, l);          // (a unit that this thread has written)
-        st_shared(sSh + off, h);
-        st_shared(sSl + off, l);
-      }
+      ok = mbar_wait(full_v, phase) && ok;
+      if (copier && more) { load_q(chunk + 1); ++n_q; }
+      __syncwarp();
+      put_weighted();
       fence_proxy_async();
-      if constexpr (NH == 2) ok = mbar_wait(bar_o, phase) && ok;     // dS takes the place of the second head's P
       __syncthreads();
-      if (warp == 0) {
+      if (warp == 0) {                                        // (in order behind the products that read the second head's P there)
         tc_fence_after();
         __syncwarp();
         issue_state();
       }
-      if (chunk + 1 < n_chunk) fetch(chunk + 1);
-      // ---- output ------------------------------------------------------------------------------------
-      ok = mbar_wait(bar_o, phase) && ok;
-      tc_fence_after();
+      // ---- output, over V --------------------------------------------------------------------------------
       const float e = fast_exp2(sm.lb[buf][mh][row].x) * a.q_scale;
       float f2 = a.q_scale, f1 = e;
       if constexpr (NORM) {
@@ -447,6 +463,8 @@ __global__ void __launch_bounds__(kThreads, 1) recurrence_tc5_kernel(const Recur
         f1 *= inv;
         f2 *= inv;
       }
+      ok = mbar_wait(bar_o, phase) && ok;
+      tc_fence_after();
 #pragma unroll
       for (int h = 0; h < 2; ++h) {
         float x[16], y[16];
@@ -457,35 +475,22 @@ __global__ void __launch_bounds__(kThreads, 1) recurrence_tc5_kernel(const Recur
         for (int u = 0; u < 2; ++u) {
           const uint32_t off = tile_off(row, cg * 4 + h * 2 + u);
           uint32_t p[4];
-          if (!NORM) {
-            const uint4 vu = ld_shared(sV + off);
-            const uint32_t vv[4] = {vu.x, vu.y, vu.z, vu.w};
+          uint4 vu = make_uint4(0, 0, 0, 0);
+          if (!NORM) vu = ld_shared(sV + off);
+          const uint32_t vv[4] = {vu.x, vu.y, vu.z, vu.w};
 #pragma unroll
-            for (int i = 0; i < 4; ++i) {
-              const float2 v = unpack2(vv[i]);
-              const int j = u * 8 + 2 * i;
-              p[i] = pack_bf162(f1 * x[j] + f2 * y[j] + skip * v.x, f1 * x[j + 1] + f2 * y[j + 1] + skip * v.y);
-            }
-          } else {
-#pragma unroll
-            for (int i = 0; i < 4; ++i) {
-              const int j = u * 8 + 2 * i;
-              p[i] = pack_bf162(f1 * x[j] + f2 * y[j], f1 * x[j + 1] + f2 * y[j + 1]);
-            }
+          for (int i = 0; i < 4; ++i) {
+            const int j = u * 8 + 2 * i;
+            float2 r = ffma2(make_float2(x[j], x[j + 1]), make_float2(f1, f1), fmul2(make_float2(y[j], y[j + 1]), make_float2(f2, f2)));
+            if (!NORM) r = ffma2(unpack2(vv[i]), make_float2(skip, skip), r);
+            p[i] = pack_bf162(r.x, r.y);
           }
-          st_shared(sQ + off, make_uint4(p[0], p[1], p[2], p[3]));   // Q is no longer read
+          st_shared(sV + off, make_uint4(p[0], p[1], p[2], p[3]));
         }
       }
+      fence_proxy_async();
     } else {
-      if (chunk + 1 < n_chunk) fetch(chunk + 1);
-      if constexpr (NORM) {
-        if (tid < N) {
-          float v = sm.n[tid] * fast_exp2(sm.dec[buf][0]);
-#pragma unroll
-          for (int w = 0; w < kThreads / 32; ++w) v += sm.n_add[w][tid];
-          sm.n[tid] = v;
-        }
-      }
+      if constexpr (NORM) advance_norm();
     }
     // ---- state ---------------------------------------------------------------------------------------
     ok = mbar_wait(bar_s, phase) && ok;
@@ -499,11 +504,38 @@ __global__ void __launch_bounds__(kThreads, 1) recurrence_tc5_kernel(const Recur
         tc_ld16(tS + h * 16u, t);
         tc_wait_ld();
 #pragma unroll
-        for (int i = 0; i < 16; ++i) S[h * 16 + i] = dc * S[h * 16 + i] + t[i];
+        for (int i = 0; i < 16; i += 2) {
+          const float2 r = ffma2(make_float2(S[h * 16 + i], S[h * 16 + i + 1]), make_float2(dc, dc), make_float2(t[i], t[i + 1]));
+          S[h * 16 + i] = r.x;
+          S[h * 16 + i + 1] = r.y;
+        }
       }
     }
-    if (warp < NH && chunk + 1 < n_chunk) put_gates(buf ^ 1);
+    if (warp < NH && more) put_gates(buf ^ 1);
     if (__syncthreads_or(ok ? 0 : 1)) break;                  // a wait ran out somewhere in the CTA
+    if constexpr (!STATE_ONLY) {
+      const int rows = n_tok - chunk * C;
+      const long long tb = t0 + (long long)chunk * C;
+      if (rows >= C) {
+        if (copier) {
+          if (NH == 2) {
+            tma_store_3d(&omap, 0, head0, (int)tb, sV);
+            tma_store_3d(&omap, 0, head0 + 1, (int)tb, sV + SLAB);
+          } else {
+            tma_store_3d(&omap, c0, head0, (int)tb, sV);
+            if (wide_v) tma_store_3d(&omap, c0 + 64, head0, (int)tb, sV + SLAB);
+          }
+          tma_store_commit();
+        }
+        __syncwarp();
+      } else {                                                // the last chunk of a sequence: its rows only
+        bf16* p = static_cast<bf16*>(a.out) + (tb + urow) * ((long long)a.heads * a.dv) + (long long)(head0 + uh) * a.dv + uc;
+#pragma unroll
+        for (int n = 0; n < 4; ++n)
+          if (uc < a.dv && urow + 32 * n < rows)
+            *reinterpret_cast<uint4*>(p + (long long)(32 * n) * a.heads * a.dv) = ld_shared(sV + tile_off(urow + 32 * n, tid & 15));
+      }
+    }
   }
   if (chunk < n_chunk) {                                      // left early: wait (bounded) for what is still in flight
     if (tid == 0) atomicOr(a.status, kStatusWaitTimeout);
@@ -514,7 +546,13 @@ __global__ void __launch_bounds__(kThreads, 1) recurrence_tc5_kernel(const Recur
     }
     mbar_wait(bar_s, phase);
   }
-  if (!STATE_ONLY && chunk == n_chunk) store_out(n_chunk - 1);
+  if (copier) {                                               // copies into and out of this CTA's shared memory
+    if (n_q > 0) mbar_wait(full_q, (uint32_t)(n_q - 1) & 1u);
+    if (n_k > 0) mbar_wait(full_k + (uint32_t)((n_k - 1) & 1) * 8u, (uint32_t)((n_k - 1) >> 1) & 1u);
+    if (n_v > 0) mbar_wait(full_v, (uint32_t)(n_v - 1) & 1u);
+    tma_store_wait_read();
+  }
+  __syncwarp();
   float* dst = STATE_ONLY ? segst : (last_seg ? cache : nullptr);
   if (dst != nullptr && row < a.dk) {
 #pragma unroll
@@ -565,13 +603,21 @@ __global__ void __launch_bounds__(256) recurrence_segment_scan_kernel(const Recu
 int tile_heads(int heads, int kv_rep, int dv, bool norm) { return !norm && dv <= 64 && kv_rep % 2 == 0 && heads % 2 == 0 ? 2 : 1; }
 
 template <int NH, bool NORM>
-cudaError_t launch_t(const RecurrenceArgs& a, cudaStream_t stream) {
+cudaError_t launch_t(const RecurrenceArgs& a, EncodeTiledFn enc, cudaStream_t stream) {
   const dim3 grid((unsigned)(a.n_seq * a.max_segs), (unsigned)(a.heads / NH), (unsigned)((a.dv + N - 1) / N));
+  const auto* x = static_cast<const bf16*>(a.qkv);
+  const int groups = a.heads / a.kv_rep;
+  CUtensorMap qmap, kmap, vmap, omap;
+  if (!make_map3(enc, &qmap, x + a.off_q, a.dk, groups, a.total, a.dk, a.stride) ||
+      !make_map3(enc, &kmap, x + a.off_k, a.dk, groups, a.total, a.dk, a.stride) ||
+      !make_map3(enc, &vmap, x + a.off_v, a.dv, a.heads, a.total, a.dv, a.stride) ||
+      !make_map3(enc, &omap, a.out, a.dv, a.heads, a.total, a.dv, (long long)a.heads * a.dv))
+    return cudaErrorInvalidValue;
   cudaError_t e;
   if (a.max_segs > 1) {
     e = cudaFuncSetAttribute(recurrence_tc5_kernel<true, NH, NORM>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem);
     if (e != cudaSuccess) return e;
-    recurrence_tc5_kernel<true, NH, NORM><<<grid, kThreads, kSmem, stream>>>(a);
+    recurrence_tc5_kernel<true, NH, NORM><<<grid, kThreads, kSmem, stream>>>(qmap, kmap, vmap, omap, a);
     e = cudaGetLastError();
     if (e != cudaSuccess) return e;
     const long long n = (long long)a.dk * a.dv + (NORM ? a.dk : 0);
@@ -581,7 +627,7 @@ cudaError_t launch_t(const RecurrenceArgs& a, cudaStream_t stream) {
   }
   e = cudaFuncSetAttribute(recurrence_tc5_kernel<false, NH, NORM>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem);
   if (e != cudaSuccess) return e;
-  recurrence_tc5_kernel<false, NH, NORM><<<grid, kThreads, kSmem, stream>>>(a);
+  recurrence_tc5_kernel<false, NH, NORM><<<grid, kThreads, kSmem, stream>>>(qmap, kmap, vmap, omap, a);
   return cudaGetLastError();
 }
 
@@ -607,10 +653,11 @@ bool recurrence_tc5_supported(const RecurrenceArgs& a) {
          (reinterpret_cast<uintptr_t>(a.state) & 15) == 0 && (a.floor == nullptr || a.skip == nullptr);
 }
 
-cudaError_t launch_recurrence_tc5(const RecurrenceArgs& a, cudaStream_t stream) {
+cudaError_t launch_recurrence_tc5(const RecurrenceArgs& a, void* encode_fn, cudaStream_t stream) {
   if (a.n_seq == 0) return cudaSuccess;
-  if (a.floor != nullptr) return launch_t<1, true>(a, stream);
-  return tile_heads(a.heads, a.kv_rep, a.dv, false) == 2 ? launch_t<2, false>(a, stream) : launch_t<1, false>(a, stream);
+  EncodeTiledFn enc = reinterpret_cast<EncodeTiledFn>(encode_fn);
+  if (a.floor != nullptr) return launch_t<1, true>(a, enc, stream);
+  return tile_heads(a.heads, a.kv_rep, a.dv, false) == 2 ? launch_t<2, false>(a, enc, stream) : launch_t<1, false>(a, enc, stream);
 }
 
 }  // namespace mixers
