@@ -116,5 +116,24 @@ __device__ __forceinline__ float gelu_tanh_f(float z) {
   return 0.5f * z * (1.f + tanhf(c * (z + 0.044715f * z * z * z)));
 }
 
+// The same for results that are rounded to T: with T = bfloat16 the hardware's exponential and reciprocal, whose errors are far below the
+// rounding.  (Below -80 the sigmoid stays at its value there, 2e-35.)
+template <typename T>
+__device__ __forceinline__ float sigmoid_t(float z) {
+  if constexpr (sizeof(T) == 2) return __fdividef(1.f, 1.f + __expf(-fmaxf(z, -80.f)));
+  else return sigmoid_f(z);
+}
+template <typename T>
+__device__ __forceinline__ float silu_t(float z) { return z * sigmoid_t<T>(z); }
+template <typename T>
+__device__ __forceinline__ float gelu_tanh_t(float z) {
+  if constexpr (sizeof(T) == 2) {
+    const float c2 = 2.f * 0.7978845608028654f;          // (1 + tanh(u)) / 2 = sigmoid(2 u)
+    return z * sigmoid_t<T>(c2 * (z + 0.044715f * z * z * z));
+  } else {
+    return gelu_tanh_f(z);
+  }
+}
+
 }  // namespace hybrid
 }  // namespace fa

@@ -9,7 +9,7 @@ namespace mixers {
 using hybrid::bf16;
 using hybrid::from_f;
 using hybrid::load_n;
-using hybrid::silu_f;
+using hybrid::silu_t;
 using hybrid::store_n;
 using hybrid::to_f;
 
@@ -160,51 +160,82 @@ __global__ void __launch_bounds__(kThreads) conv_silu_kernel(const ConvArgs a) {
       for (int i = 0; i < VEC; ++i) v[i] = 0.f;
     }
   };
-  constexpr int W = TAPS > 0 ? TAPS : 1;
-  float win[W][VEC], wk[W][VEC];             // win[k]: the input k positions back
+  auto emit = [&](long long t, float (&acc)[VEC]) {
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) acc[i] = silu_t<T>(acc[i]);
+    store_n<VEC>(static_cast<T*>(a.out) + t * a.channels + c, acc);
+  };
   if constexpr (TAPS > 0) {
+    float win[TAPS][VEC], wk[TAPS][VEC];     // win[k]: the input k positions back
 #pragma unroll
     for (int k = 0; k < TAPS; ++k) load_n<VEC>(wt + (long long)(TAPS - 1 - k) * a.channels, wk[k]);
-  }
-  int seq = -1;
-  for (long long t = ta; t < tb; ++t) {
-    const int s = a.tok_seq[t], pos = a.positions[t];
-    if (s < 0 || s >= a.n_seq) {
-      if (c == 0) atomicOr(a.status, 2);
-      continue;
-    }
-    const long long seq0 = a.cu != nullptr ? a.cu[s] : t;
-    float acc[VEC];
+    auto advance = [&](long long t, const float (&in)[VEC]) {
+      float acc[VEC];
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) acc[i] = bias[i];
-    if constexpr (TAPS > 0) {
-      if (s == seq) {
+      for (int k = TAPS - 1; k > 0; --k)
 #pragma unroll
-        for (int k = TAPS - 1; k > 0; --k)
+        for (int i = 0; i < VEC; ++i) win[k][i] = win[k - 1][i];
 #pragma unroll
-          for (int i = 0; i < VEC; ++i) win[k][i] = win[k - 1][i];
-      } else {
-#pragma unroll
-        for (int k = 1; k < TAPS; ++k) input(t, k, s, pos, seq0, win[k]);
+      for (int i = 0; i < VEC; ++i) {
+        win[0][i] = in[i];
+        acc[i] = bias[i];
       }
-      load_n<VEC>(z + t * a.stride, win[0]);
 #pragma unroll
       for (int k = 0; k < TAPS; ++k)
 #pragma unroll
         for (int i = 0; i < VEC; ++i) acc[i] += wk[k][i] * win[k][i];
-    } else {
-      for (int k = 0; k < taps; ++k) {
-        float w[VEC];
-        load_n<VEC>(wt + (long long)(taps - 1 - k) * a.channels, w);
-        input(t, k, s, pos, seq0, win[0]);
+      emit(t, acc);
+    };
+    int seq = -1;
+    for (long long t = ta; t < tb;) {
+      const int s = a.tok_seq[t], pos = a.positions[t];
+      if (s < 0 || s >= a.n_seq) {
+        if (c == 0) atomicOr(a.status, 2);
+        seq = -1;
+        ++t;
+        continue;
+      }
+      if (s != seq) {                        // win[k] will be k + 1 positions back
+        const long long seq0 = a.cu != nullptr ? a.cu[s] : t;
 #pragma unroll
-        for (int i = 0; i < VEC; ++i) acc[i] += w[i] * win[0][i];
+        for (int k = 1; k < TAPS; ++k) input(t, k, s, pos, seq0, win[k - 1]);
+        seq = s;
+      }
+      constexpr int B = 4;                   // tokens whose inputs are fetched together
+      if (t + B <= tb && a.tok_seq[t + B - 1] == s) {
+        float in[B][VEC];
+#pragma unroll
+        for (int j = 0; j < B; ++j) load_n<VEC>(z + (t + j) * a.stride, in[j]);
+#pragma unroll
+        for (int j = 0; j < B; ++j) advance(t + j, in[j]);
+        t += B;
+      } else {
+        float in[VEC];
+        load_n<VEC>(z + t * a.stride, in);
+        advance(t, in);
+        ++t;
       }
     }
-    seq = s;
+  } else {
+    for (long long t = ta; t < tb; ++t) {
+      const int s = a.tok_seq[t], pos = a.positions[t];
+      if (s < 0 || s >= a.n_seq) {
+        if (c == 0) atomicOr(a.status, 2);
+        continue;
+      }
+      const long long seq0 = a.cu != nullptr ? a.cu[s] : t;
+      float acc[VEC];
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) acc[i] = silu_f(acc[i]);
-    store_n<VEC>(static_cast<T*>(a.out) + t * a.channels + c, acc);
+      for (int i = 0; i < VEC; ++i) acc[i] = bias[i];
+      for (int k = 0; k < a.taps; ++k) {
+        float w[VEC], in[VEC];
+        load_n<VEC>(wt + (long long)(a.taps - 1 - k) * a.channels, w);
+        input(t, k, s, pos, seq0, in);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) acc[i] += w[i] * in[i];
+      }
+      emit(t, acc);
+    }
   }
 }
 

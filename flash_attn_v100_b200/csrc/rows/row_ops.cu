@@ -148,10 +148,10 @@ __global__ void __launch_bounds__(kThreads) residual_norm_kernel(const ResidualN
 
 // Gated norm of row `blockIdx.x`, part `blockIdx.y` of `a.group` columns, one CTA each.  SILU: out = rmsnorm(o * silu(g)) * w,
 // otherwise out = rmsnorm(o) * w * sigmoid(g).
-template <bool SILU>
-__device__ __forceinline__ float gate_first(float o, float g) { return SILU ? o * silu_f(g) : o; }
-template <bool SILU>
-__device__ __forceinline__ float gate_last(float y, float g) { return SILU ? y : y * sigmoid_f(g); }
+template <typename T, bool SILU>
+__device__ __forceinline__ float gate_first(float o, float g) { return SILU ? o * silu_t<T>(g) : o; }
+template <typename T, bool SILU>
+__device__ __forceinline__ float gate_last(float y, float g) { return SILU ? y : y * sigmoid_t<T>(g); }
 
 template <typename T, int VEC, int KEEP, bool SILU>
 __global__ void __launch_bounds__(kThreads) gated_norm_kernel(const GatedNormArgs a) {
@@ -171,7 +171,7 @@ __global__ void __launch_bounds__(kThreads) gated_norm_kernel(const GatedNormArg
       float gv[VEC];
       load_n<VEC>(g + c * VEC, gv);
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) v[i] = gate_first<SILU>(v[i], gv[i]);
+      for (int i = 0; i < VEC; ++i) v[i] = gate_first<T, SILU>(v[i], gv[i]);
     }
   };
   if constexpr (KEEP > 0) {
@@ -197,7 +197,7 @@ __global__ void __launch_bounds__(kThreads) gated_norm_kernel(const GatedNormArg
     load_n<VEC>(w + c * VEC, wv);
     if constexpr (!SILU) load_n<VEC>(g + c * VEC, gv);
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) v[i] = gate_last<SILU>(v[i] * inv * wv[i], SILU ? 0.f : gv[i]);
+    for (int i = 0; i < VEC; ++i) v[i] = gate_last<T, SILU>(v[i] * inv * wv[i], SILU ? 0.f : gv[i]);
     store_n<VEC>(out + c * VEC, v);
   };
   if constexpr (KEEP > 0) {
@@ -214,38 +214,52 @@ __global__ void __launch_bounds__(kThreads) gated_norm_kernel(const GatedNormArg
   }
 }
 
-// The same for parts of at most 256 columns (a multiple of 8): LANES lanes per (row, part).
-template <typename T, int LANES, bool SILU>
+// The same for parts of at most LANES * KEEP * 8 columns (a multiple of 8): LANES lanes per (row, part), KEEP vectors each.
+template <typename T, int LANES, int KEEP, bool SILU>
 __global__ void __launch_bounds__(kThreads) gated_norm_small_kernel(const GatedNormArgs a, const long long parts) {
   constexpr int VEC = 8;
   const long long part = ((long long)blockIdx.x * kThreads + threadIdx.x) / LANES;
-  const int c = (threadIdx.x % LANES) * VEC;
+  const int lane = threadIdx.x % LANES;
   const int per_row = a.cols / a.group;
-  const bool live = part < parts && c < a.group;
+  const bool live = part < parts;
   const long long row = live ? part / per_row : 0;
-  const int col = live ? (int)(part - row * per_row) * a.group + c : 0;
-  float v[VEC], gv[VEC];
-#pragma unroll
-  for (int i = 0; i < VEC; ++i) v[i] = 0.f;
+  const int c0 = live ? (int)(part - row * per_row) * a.group : 0;
+  const T* o = static_cast<const T*>(a.o) + row * a.cols + c0;
+  const T* g = static_cast<const T*>(a.g) + row * a.g_stride + c0;
+  float v[KEEP][VEC], gv[KEEP][VEC];
   float ss = 0.f;
-  if (live) {
-    load_n<VEC>(static_cast<const T*>(a.o) + row * a.cols + col, v);
-    load_n<VEC>(static_cast<const T*>(a.g) + row * a.g_stride + col, gv);
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) {
-      v[i] = gate_first<SILU>(v[i], gv[i]);
-      ss += v[i] * v[i];
+  for (int n = 0; n < KEEP; ++n) {
+    const int c = (lane + n * LANES) * VEC;
+    if (live && c < a.group) {
+      load_n<VEC>(o + c, v[n]);
+      load_n<VEC>(g + c, gv[n]);
+    }
+  }
+#pragma unroll
+  for (int n = 0; n < KEEP; ++n) {
+    if (live && (lane + n * LANES) * VEC < a.group) {
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) {
+        v[n][i] = gate_first<T, SILU>(v[n][i], gv[n][i]);
+        ss += v[n][i] * v[n][i];
+      }
     }
   }
 #pragma unroll
   for (int o = LANES / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
   if (!live) return;
   const float inv = 1.f / sqrtf(ss / (float)a.group + a.eps);
-  float wv[VEC];
-  load_n<VEC>(static_cast<const T*>(a.w) + col, wv);
 #pragma unroll
-  for (int i = 0; i < VEC; ++i) v[i] = gate_last<SILU>(v[i] * inv * wv[i], gv[i]);
-  store_n<VEC>(static_cast<T*>(a.out) + row * a.out_stride + col, v);
+  for (int n = 0; n < KEEP; ++n) {
+    const int c = (lane + n * LANES) * VEC;
+    if (c >= a.group) break;
+    float wv[VEC];
+    load_n<VEC>(static_cast<const T*>(a.w) + c0 + c, wv);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[n][i] = gate_last<T, SILU>(v[n][i] * inv * wv[i], gv[n][i]);
+    store_n<VEC>(static_cast<T*>(a.out) + row * a.out_stride + c0 + c, v[n]);
+  }
 }
 
 // gu [rows, 2n] (gate, then linear branch): out = g sigmoid(alpha g) (u + shift), g = min(gate, limit),
@@ -301,7 +315,7 @@ __global__ void __launch_bounds__(kThreads) gelu_kernel(const T* z, long long z_
     float v[VEC];
     load_n<VEC>(z + row * z_stride + c, v);
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) v[j] = gelu_tanh_f(v[j]);
+    for (int j = 0; j < VEC; ++j) v[j] = gelu_tanh_t<T>(v[j]);
     store_n<VEC>(out + row * out_stride + c, v);
   }
 }
@@ -372,9 +386,11 @@ static void launch_gated_norm_t(const GatedNormArgs& a, cudaStream_t s) {
   const dim3 grid((unsigned)a.rows, (unsigned)(a.cols / a.group));
   const long long parts = a.rows * (a.cols / a.group);
   auto blocks = [&](int lanes) { return (unsigned)((parts * lanes + kThreads - 1) / kThreads); };
-  if (vec && a.group <= 64) gated_norm_small_kernel<T, 8, SILU><<<blocks(8), kThreads, 0, s>>>(a, parts);
-  else if (vec && a.group <= 128) gated_norm_small_kernel<T, 16, SILU><<<blocks(16), kThreads, 0, s>>>(a, parts);
-  else if (vec && a.group <= 256) gated_norm_small_kernel<T, 32, SILU><<<blocks(32), kThreads, 0, s>>>(a, parts);
+  if (vec && a.group <= 64) gated_norm_small_kernel<T, 8, 1, SILU><<<blocks(8), kThreads, 0, s>>>(a, parts);
+  else if (vec && a.group <= 128) gated_norm_small_kernel<T, 8, 2, SILU><<<blocks(8), kThreads, 0, s>>>(a, parts);
+  else if (vec && a.group <= 256) gated_norm_small_kernel<T, 16, 2, SILU><<<blocks(16), kThreads, 0, s>>>(a, parts);
+  else if (vec && a.group <= 512) gated_norm_small_kernel<T, 32, 2, SILU><<<blocks(32), kThreads, 0, s>>>(a, parts);
+  else if (vec && a.group <= 1024) gated_norm_small_kernel<T, 32, 4, SILU><<<blocks(32), kThreads, 0, s>>>(a, parts);
   else if (vec && a.group <= 8 * kThreads) gated_norm_kernel<T, 8, 1, SILU><<<grid, kThreads, 0, s>>>(a);
   else if (vec && a.group <= 16 * kThreads) gated_norm_kernel<T, 8, 2, SILU><<<grid, kThreads, 0, s>>>(a);
   else if (vec && a.group <= 32 * kThreads) gated_norm_kernel<T, 8, 4, SILU><<<grid, kThreads, 0, s>>>(a);

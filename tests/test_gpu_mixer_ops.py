@@ -292,7 +292,7 @@ def test_convolution_in_portions(channels, taps, dtype):
 
 
 @pytest.mark.parametrize("dtype", TYPES)
-@pytest.mark.parametrize("H, K, V", [(4, 32, 48), (2, 128, 256), (3, 20, 12), (1, 300, 8), (5, 64, 64)])
+@pytest.mark.parametrize("H, K, V", [(4, 32, 48), (2, 128, 256), (3, 20, 12), (1, 300, 8), (5, 64, 64), (2, 9, 16), (640, 8, 8)])
 def test_max_gate_step_equals_the_scan(H, K, V, dtype):
     """Decode steps in one kernel: many tokens one by one, from position 0 in slots with leftovers."""
     g, T, cap = gen(H * K), 12, 9.0
@@ -323,7 +323,7 @@ def test_max_gate_step_equals_the_scan(H, K, V, dtype):
 
 
 @pytest.mark.parametrize("dtype", TYPES)
-@pytest.mark.parametrize("H, G, N, V, taps", [(4, 2, 32, 32, 4), (6, 1, 128, 64, 4), (2, 2, 20, 12, 3), (3, 3, 64, 200, 2), (8, 2, 16, 16, 1)])
+@pytest.mark.parametrize("H, G, N, V, taps", [(4, 2, 32, 32, 4), (6, 1, 128, 64, 4), (2, 2, 20, 12, 3), (3, 3, 64, 200, 2), (8, 2, 16, 16, 1), (4, 1, 9, 8, 6), (1280, 160, 8, 8, 4)])
 def test_ssd_step_equals_the_scan(H, G, N, V, taps, dtype):
     g, T = gen(H * N), 11
     ch = H * V + 2 * G * N
