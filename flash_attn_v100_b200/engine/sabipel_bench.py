@@ -28,7 +28,7 @@ def sabipel_config() -> HybridConfig:
     attention = ChunkedAttentionSpec(HEADS, KV_HEADS, DIM, DIM, DIM ** -0.5, CHUNK, power_of_two_slopes(HEADS), True)
     order = (memory, SSD, SSD, attention) * (hb.LAYERS // 4)
     return HybridConfig(VOCAB, WIDTH, tuple(HybridLayer(m, GeluSpec(FF)) for m in order), 1e-6, parallel=True, embed_scale=4.0,
-                        bigram=BigramSpec(BUCKETS, 31, 7), max_positions=16384)
+                        bigram=BigramSpec(BUCKETS, 8191, 131), max_positions=16384)
 
 
 def kernel_records(device, steps, warmup, peaks, which="all"):
@@ -90,7 +90,7 @@ def kernel_records(device, steps, warmup, peaks, which="all"):
         pos, seq = torch.arange(per, dtype=torch.int32, device=device).repeat(n_seq), rows.repeat_interleave(per).contiguous()
         tok = torch.randint(0, VOCAB, (T,), generator=g, device=device)
         last = torch.zeros(n_seq, dtype=torch.int32, device=device)
-        add("bigram_rows", "sabipel", label, lambda: rops.bigram_rows(tok, starts, rows, last, BUCKETS, 31, 7, st, cu_seqlens=seqs.cu_seqlens), T * 12)
+        add("bigram_rows", "sabipel", label, lambda: rops.bigram_rows(tok, starts, rows, last, BUCKETS, 8191, 131, st, cu_seqlens=seqs.cu_seqlens), T * 12)
         blocks = (per + 15) // 16
         table = torch.arange(n_seq * blocks, dtype=torch.int32, device=device).view(n_seq, blocks)
         kp, vp = (torch.zeros(n_seq * blocks, KV_HEADS, 16, DIM, dtype=torch.bfloat16, device=device) for _ in range(2))

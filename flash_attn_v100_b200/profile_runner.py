@@ -18,13 +18,15 @@ def main():
     ap.add_argument("--case", default="paged_decode",
                     choices=["paged_decode", "int8_decode", "varlen_prefill", "contig_decode", "int8_kv_decode",
                              "sliding_window_decode", "latent_decode", "latent_prefill", "lightning_prefill",
-                             "lightning_decode"])
+                             "lightning_decode", "memory_prefill", "ssd_prefill", "memory_decode", "ssd_decode", "kv_prefill", "kv_decode"])
     ap.add_argument("--batch", type=int, default=16)
     ap.add_argument("--iters", type=int, default=3)
     ap.add_argument("--seed", type=int, default=0)
     args = ap.parse_args()
     if args.case.startswith(("latent", "lightning")):
         return hybrid(args)
+    if args.case.startswith(("memory", "ssd", "kv")):
+        return mixers(args)
     import flash_attn_v100 as fa
     import flash_attn_v100_b200
     from flash_attn_v100_b200.synthetic import make_paged_tables
@@ -124,6 +126,60 @@ def hybrid(args):
         starts = torch.full((B,), 0 if prompt else 9, dtype=torch.int32, device=dev)
         run = lambda: hops.lightning(z, (0, H * D, 2 * H * D), H, D, D, decay, state, rows, starts, st, cu_seqlens=cu, max_len=n)
         print(f"case {args.case}: seqs={B} row_bytes={B * n * H * D * 8} state_bytes={B * H * D * D * 8}")
+    for _ in range(args.iters + 1):
+        run()
+    torch.cuda.synchronize()
+    if int(st.item()):
+        raise RuntimeError(f"a kernel recorded status {int(st.item())}")
+    print("done")
+
+
+def mixers(args):
+    """Kernels of the Sabipel decoder: 32 heads of 128 with a normaliser, 64 state-space heads of 64 in 8 groups with a state of 128, 32
+    query heads on 8 of 128; prompts of 1024 and 4096 cached tokens."""
+    from flash_attn_v100_b200 import mixer_ops as mops
+    dev = torch.device("cuda", 0)
+    g = torch.Generator(device=dev).manual_seed(args.seed)
+    rnd = lambda *s: torch.randn(*s, generator=g, device=dev).bfloat16()
+    f32 = lambda *s: torch.rand(*s, generator=g, device=dev)
+    st = torch.zeros(1, dtype=torch.int32, device=dev)
+    B, D = args.batch, 128
+    rows = torch.arange(B, dtype=torch.int32, device=dev)
+    kind, prompt = args.case.split("_")[0], args.case.endswith("prefill")
+    n = 1024 if prompt else 1
+    T, cu = B * n, torch.arange(B + 1, dtype=torch.int32, device=dev) * n
+    seqs = mops.Sequences(rows, torch.full((B,), 0 if prompt else 9, dtype=torch.int32, device=dev), cu if prompt else None, n)
+    if kind == "kv":
+        H, G, ctx = 32, 8, 4096
+        q, gate, slopes = rnd(T, H * D), rnd(T, H * D), f32(H)
+        if prompt:
+            k, v = rnd(T, G * D), rnd(T, G * D)
+            run = lambda: mops.kv_prefill(q, k, v, cu, cu, n, H, G, D ** -0.5, slopes, st, gate=gate)
+            print(f"case kv_prefill: seqs={B} flops={B * 4 * H * D * n * (n + 1) // 2}")
+        else:
+            table = torch.randperm(B * ctx // 16).to(torch.int32).view(B, ctx // 16).to(dev)
+            pages = mops.Pages(rnd(B * ctx // 16, G, 16, D), rnd(B * ctx // 16, G, 16, D), table, rows, torch.full((B,), ctx - 1, dtype=torch.int32, device=dev), st)
+            run = lambda: mops.kv_attention(pages, q, H, ctx, D ** -0.5, slopes=slopes, gate=gate)
+            print(f"case kv_decode: B={B} tokens={B * ctx} cache_bytes={B * ctx * G * D * 4}")
+    else:
+        H, G, dv = (32, 32, D) if kind == "memory" else (64, 8, 64)
+        hv, gk = H * dv, G * D
+        state = torch.zeros(B, H, D, dv, device=dev)
+        norm, m = torch.zeros(B, 2, H, D, device=dev), torch.zeros(B, 2, H, device=dev)
+        la, b = -0.1 * f32(H, T), f32(H, T)
+        extra = dict(floor=b + 0.5, n0=torch.zeros(B, H, D, device=dev), norm=norm, norm_eps=1e-6) if kind == "memory" else dict(skip=f32(H))
+        if prompt:
+            x = rnd(T, hv + 2 * gk)
+            run = lambda: mops.recurrence(x, (hv + gk, hv, 0), H, G, D, dv, la, b, state, seqs, st, **extra)
+        elif kind == "memory":
+            x = rnd(T, hv + 2 * gk + 2 * H)
+            run = lambda: mops.max_gate_step(x, (hv + gk, hv, 0), H, D, dv, hv + 2 * gk, hv + 2 * gk + H, rnd(H), rnd(H), 15.0, state, norm, m, seqs, st,
+                                             q_scale=D ** -0.5, norm_eps=1e-6)
+        else:
+            x, ring, w, cb = rnd(T, hv + 2 * gk + H), rnd(B, 4, hv + 2 * gk), rnd(4, hv + 2 * gk), rnd(hv + 2 * gk)
+            bias, a_log, skip = f32(H), f32(H), f32(H)
+            run = lambda: mops.ssd_step(x, 0, H, G, D, dv, hv + 2 * gk, bias, a_log, skip, w, cb, ring, state, seqs, st)
+        print(f"case {args.case}: seqs={B} row_bytes={T * (2 * hv + 2 * gk) * 2} state_bytes={B * H * D * dv * 8}")
     for _ in range(args.iters + 1):
         run()
     torch.cuda.synchronize()

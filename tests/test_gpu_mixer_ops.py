@@ -323,7 +323,7 @@ def test_max_gate_step_equals_the_scan(H, K, V, dtype):
 
 
 @pytest.mark.parametrize("dtype", TYPES)
-@pytest.mark.parametrize("H, G, N, V, taps", [(4, 2, 32, 32, 4), (6, 1, 128, 64, 4), (2, 2, 20, 12, 3), (3, 3, 64, 200, 2), (8, 2, 16, 16, 1), (4, 1, 9, 8, 6), (1280, 160, 8, 8, 4)])
+@pytest.mark.parametrize("H, G, N, V, taps", [(4, 2, 40, 32, 4), (6, 1, 128, 64, 4), (2, 2, 20, 12, 3), (3, 3, 64, 200, 2), (8, 2, 16, 16, 1), (4, 1, 9, 8, 6), (1280, 160, 8, 8, 4)])
 def test_ssd_step_equals_the_scan(H, G, N, V, taps, dtype):
     g, T = gen(H * N), 11
     ch = H * V + 2 * G * N
@@ -388,7 +388,7 @@ def attend(q, k, v, pos, chunk, scale, slopes, gate):
     return o * orc.sigmoid(gate.double()) if gate is not None else o
 
 
-ATTENTION_SIZES = [(4, 1, 64, 32), (8, 2, 128, 128), (16, 1, 64, 64), (24, 1, 48, 72), (3, 3, 32, 128), (6, 2, 10, 14), (2, 1, 160, 24)]
+ATTENTION_SIZES = [(4, 1, 56, 32), (8, 2, 128, 128), (16, 1, 64, 64), (24, 1, 48, 72), (3, 3, 32, 128), (6, 2, 10, 14), (2, 1, 160, 24)]
 
 
 @pytest.mark.parametrize("dtype", TYPES)
@@ -436,7 +436,7 @@ def test_one_long_row_is_shared_by_several_blocks():
         assert int(st.item()) == 0
 
 
-@pytest.mark.parametrize("H, G, K, V", [(4, 1, 64, 32), (8, 2, 128, 128), (3, 3, 32, 128), (6, 2, 128, 64), (2, 1, 40, 24)])
+@pytest.mark.parametrize("H, G, K, V", [(4, 1, 56, 32), (8, 2, 128, 128), (3, 3, 32, 128), (6, 2, 128, 64), (2, 1, 40, 24), (2, 1, 64, 48)])
 def test_prompt_attention(H, G, K, V):
     """Pieces whose queries are all or only the last of their keys; a strong far key; steep and flat slopes."""
     g = gen(H * K)
